@@ -30,6 +30,12 @@ def libpath():
 
 
 @pytest.fixture(scope="session")
+def float_libpath():
+    b = importlib.import_module(PKG + ".build")
+    return b.build(library=b.FLOAT_LIBRARY)
+
+
+@pytest.fixture(scope="session")
 def kmod(libpath):
     """The drop-in kernel module (needs the built library; GPU needed only to call it)."""
     return importlib.import_module(PKG + ".kernel")

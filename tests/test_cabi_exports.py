@@ -14,16 +14,11 @@ REFERENCE_SYMBOLS = [
 ]
 
 
-def declared_functions():
-    names = []
-    for fn in sorted(os.listdir(os.path.join(ROOT, "include"))):
-        if not fn.endswith(".h"):
-            continue
-        src = open(os.path.join(ROOT, "include", fn)).read()
-        src = re.sub(r"/\*.*?\*/", "", src, flags=re.S)
-        src = re.sub(r"^\s*#.*$", "", src, flags=re.M)
-        names += re.findall(r"\b([A-Za-z_][A-Za-z0-9_]*)\s*\([^;{]*\)\s*;", src)
-    return names
+def declared_functions(header="zkds_int64.h"):
+    src = open(os.path.join(ROOT, "include", header)).read()
+    src = re.sub(r"/\*.*?\*/", "", src, flags=re.S)
+    src = re.sub(r"^\s*#.*$", "", src, flags=re.M)
+    return re.findall(r"\b([A-Za-z_][A-Za-z0-9_]*)\s*\([^;{]*\)\s*;", src)
 
 
 def test_header_declares_the_reference_symbols():
@@ -38,6 +33,15 @@ def test_library_exports_every_declared_symbol(libpath):
     assert len(names) >= len(REFERENCE_SYMBOLS) + 10
     missing = [n for n in names if not hasattr(lib, n)]
     assert not missing, missing
+
+
+def test_float_library_exports_every_declared_symbol(float_libpath):
+    lib = ctypes.CDLL(float_libpath)
+    names = declared_functions("zkds_float.h")
+    assert len(names) >= 10
+    missing = [n for n in names if not hasattr(lib, n)]
+    assert not missing, missing
+    assert sorted(os.listdir(os.path.join(ROOT, "include"))) == ["zkds_float.h", "zkds_int64.h"]
 
 
 def test_host_only_entry_points(libpath, orc):

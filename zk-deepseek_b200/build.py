@@ -1,11 +1,16 @@
-"""Builds libint64gemm.so for sm_100a with nvcc, in-tree, beside this file.
+"""Builds the CUDA libraries for sm_100a with nvcc, in-tree, beside this file.
 
-    python zk-deepseek_b200/build.py [--force] [--verbose]
+    python zk-deepseek_b200/build.py [--force] [--verbose] [NAME ...]
 
-nvcc cross-compiles without a GPU.  The library links the CUDA runtime statically
-and resolves the driver entry points it needs (tensor-map encoding) at run time, so
-it loads on a machine without a GPU as well.
+    libint64gemm.so   the int64 fixed-point kernels of the integer model
+    libfloatops.so    the kernels of the floating-point decoder designs
+
+nvcc cross-compiles without a GPU.  The libraries link the CUDA runtime statically and resolve the driver entry
+points they need (tensor-map encoding) at run time, so they load on a machine without a GPU as well.  A library is
+compiled when it is missing or older than one of its sources; callers on a fresh checkout build only the one they
+load.
 """
+import fcntl
 import os
 import shutil
 import subprocess
@@ -13,38 +18,80 @@ import sys
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
-OUT = os.path.join(HERE, "libint64gemm.so")
-SOURCES = ["capi.cu", "fixedpoint.cu", "gemm_exact.cu", "limb_gemm.cu", "converters.cu"]
+INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-         "-Xcompiler", "-fPIC", "-shared"]
+         "-Xcompiler", "-fPIC"]
+# library -> (translation units, headers)
+LIBRARIES = {
+    "libint64gemm.so": (["capi.cu", "fixedpoint.cu", "gemm_exact.cu", "limb_gemm.cu", "converters.cu"],
+                        ["common.cuh", "kernels.h", "tcgen05.cuh", "zkds_int64.h"]),
+    "libfloatops.so": (["float_capi.cu", "float_ops.cu", "float_gemm.cu", "float_gemm_tc.cu", "float_attention.cu"],
+                       ["common.cuh", "float_common.cuh", "tcgen05.cuh", "zkds_float.h"]),
+}
+INT_LIBRARY, FLOAT_LIBRARY = "libint64gemm.so", "libfloatops.so"
+OUT = os.path.join(HERE, INT_LIBRARY)
 
 
-def _stale():
-    if not os.path.exists(OUT):
+def _dep(name):
+    path = os.path.join(CSRC, name)
+    return path if os.path.exists(path) else os.path.join(INCLUDE, name)
+
+
+def _stale(library):
+    out = os.path.join(HERE, library)
+    if not os.path.exists(out):
         return True
-    t = os.path.getmtime(OUT)
-    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)]
-    deps.append(os.path.join(os.path.dirname(HERE), "include", "zkds_int64.h"))
-    return any(os.path.getmtime(d) > t for d in deps)
+    t = os.path.getmtime(out)
+    sources, headers = LIBRARIES[library]
+    return any(os.path.getmtime(_dep(d)) > t for d in sources + headers)
 
 
-def build(force=False, verbose=False):
-    if not force and not _stale():
-        return OUT
+def _compile(library, verbose):
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
-    tmp = OUT + ".partial"          # the library appears under its name only once it is complete
-    cmd = [nvcc] + FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-o", tmp] + \
-          [os.path.join(CSRC, s) for s in SOURCES]
-    res = subprocess.run(cmd, capture_output=True, text=True)
-    if verbose or res.returncode != 0:
-        sys.stderr.write(res.stdout + res.stderr)
-    if res.returncode != 0:
-        if os.path.exists(tmp):
-            os.remove(tmp)
-        raise RuntimeError("nvcc failed building libint64gemm.so")
-    os.replace(tmp, OUT)
-    return OUT
+    out = os.path.join(HERE, library)
+    tag = ".%d.partial" % os.getpid()
+    flags = FLAGS + (["-Xptxas", "-v"] if verbose else [])
+    objs, jobs, failed = [], [], False
+    for src in LIBRARIES[library][0]:                  # the translation units compile side by side
+        obj = os.path.join(HERE, src + tag + ".o")
+        objs.append(obj)
+        jobs.append(subprocess.Popen([nvcc] + flags + ["-x", "cu", "-c", os.path.join(CSRC, src), "-o", obj],
+                                     stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True))
+    for job in jobs:
+        text = job.communicate()[0]
+        if verbose or job.returncode:
+            sys.stderr.write(text)
+        failed |= job.returncode != 0
+    try:
+        if not failed:
+            # the library appears under its name only once it is complete
+            res = subprocess.run([nvcc] + FLAGS[:2] + ["-shared", "-Xcompiler", "-fPIC", "-o", out + tag] + objs,
+                                 capture_output=True, text=True)
+            failed = res.returncode != 0
+            if failed:
+                sys.stderr.write(res.stdout + res.stderr)
+        if failed:
+            raise RuntimeError("nvcc failed building " + library)
+        os.replace(out + tag, out)
+    finally:
+        for f in objs + [out + tag]:
+            if os.path.exists(f):
+                os.remove(f)
+    return out
+
+
+def build(force=False, verbose=False, library=INT_LIBRARY):
+    out = os.path.join(HERE, library)
+    if not force and not _stale(library):
+        return out
+    with open(out + ".lock.partial", "w") as lock:     # one process compiles, the others wait for it
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if force or _stale(library):
+            _compile(library, verbose)
+    return out
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv))
+    names = [a for a in sys.argv[1:] if not a.startswith("-")] or list(LIBRARIES)
+    for name in names:
+        print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv, library=name))

@@ -1,4 +1,5 @@
-"""Token generation over the integer model with every layer resident on the GPU.
+"""Token generation with every layer resident on the GPU: the loop that serves the integer model and the
+floating-point decoder designs, and the command line.
 
 Follows the loop of the reference's `generate()` (inference/generate.py:164-286): the prompt
 is run as one prefill, then one position per step; `prompt_mask` keeps prompt tokens from being
@@ -15,15 +16,19 @@ Differences, all on the host side of the hot path:
   * `sample()` in the reference has its stochastic branch switched off (`sample_open = False`,
     generate.py:80) and returns the argmax for every temperature; the same is done here.
 """
+import argparse
+import importlib
+import json
 import os
+import sys
 from typing import List, Optional
 
 import torch
 
-try:
-    from . import model as M
-except ImportError:  # pragma: no cover - drop-in use with this directory first on sys.path
-    import model as M
+
+def _module(name):
+    # drop-in use: this directory first on sys.path, no package
+    return importlib.import_module("." + name, __package__) if __package__ else importlib.import_module(name)
 
 
 def load_resident(ckpt_path: str, args, device="cuda", cache_batch: int = 1, prepare: bool = True):
@@ -34,6 +39,7 @@ def load_resident(ckpt_path: str, args, device="cuda", cache_batch: int = 1, pre
     host and rebuilds one `Block` at a time; here all of them stay resident, and with `prepare` the limb
     planes of every static weight are built once at load instead of at first use."""
     from safetensors.torch import load_file, load_model
+    M = _module("model")
     with torch.device(device):
         model = M.Transformer(args)
     load_model(model.embed, os.path.join(ckpt_path, "embed_int.safetensors"))
@@ -61,30 +67,19 @@ def sample(logits: torch.Tensor, temperature: float = 1.0) -> torch.Tensor:
     return logits.argmax(dim=-1)
 
 
-def _forward_step(model, toks, prev_pos, layer_probe):
-    """one pass over all layers; finish_inference raises ZkdsError if a kernel flagged its operands"""
-    h, start_pos, seqlen = model.prep_inference(toks, prev_pos)
-    layer_tokens = []
-    for i in range(model.args.n_layers):
-        h = model.layer_inference(i, h, start_pos, seqlen)
-        if layer_probe:
-            probe = model.head(model.norm(h)[0][:, -1].contiguous()[None, :])
-            layer_tokens.append(probe.argmax(dim=-1).view(-1).tolist())
-    return model.finish_inference(h), layer_tokens
-
-
 @torch.inference_mode()
 def generate(model, prompt_tokens: List[List[int]], max_new_tokens: int, eos_id: int,
              temperature: float = 1.0, layer_probe: bool = False,
              trace: Optional[list] = None) -> List[List[int]]:
     """Returns the completion tokens of every prompt (generate.py:164-286).
 
-    model: a `Transformer` whose `layers[i]` are loaded `Block`s (caches sized for the batch).
+    model: what `registry.load` returns: a `Transformer` whose `layers[i]` are loaded `Block`s (caches sized for
+    the batch), or a `FloatTransformer`.  The loop only uses begin_batch / step / end_batch, `args` and `device`.
     trace: optional list; receives one dict per step (`pos`, `next_token`, and `layer_tokens` when
     `layer_probe` is set) in place of the reference's progress prints.
     """
     args = model.args
-    device = model.freqs_cis.device
+    device = model.device
     prompt_lens = [len(t) for t in prompt_tokens]
     assert max(prompt_lens) <= args.max_seq_len, \
         f"Prompt length exceeds model maximum sequence length (max_seq_len={args.max_seq_len})"
@@ -95,36 +90,21 @@ def generate(model, prompt_tokens: List[List[int]], max_new_tokens: int, eos_id:
     prev_pos = 0
     finished = torch.zeros(len(prompt_tokens), dtype=torch.bool, device=device)
     prompt_mask = tokens != -1
-    for cur_pos in range(min(prompt_lens), total_len):
-        if M.snark:
-            os.makedirs(f"{M.zkDataDir}/pos_{prev_pos}", exist_ok=True)
-            M.saveTensor(f"{M.zkDataDir}/pos_{prev_pos}/tokens.bin", tokens[0][prev_pos:cur_pos].cpu())
-        rerun = False
-        try:
-            logits, layer_tokens = _forward_step(model, tokens[:, prev_pos:cur_pos], prev_pos, layer_probe)
-        except M.K.ZkdsError as err:
-            if err.status != M.K.ERR_RANGE:
-                raise
-            # an activation exceeded the limb bound promised for it (M.ACT_LIMBS, MLA.score_limbs): that
-            # pass's numbers are wrong.  The step only wrote cache rows it owns, so it is simply run again
-            # with every limb count measured on the device.
-            with M.measured_limbs(model):
-                logits, layer_tokens = _forward_step(model, tokens[:, prev_pos:cur_pos], prev_pos, layer_probe)
-            rerun = True
-        next_token = (sample(logits, temperature) if temperature > 0 else logits.argmax(dim=-1)).view(-1)
-        next_token = torch.where(prompt_mask[:, cur_pos], tokens[:, cur_pos], next_token)
-        tokens[:, cur_pos] = next_token
-        finished |= torch.logical_and(~prompt_mask[:, cur_pos], next_token == eos_id)
-        prev_pos = cur_pos
-        if trace is not None:
-            step = {"pos": cur_pos, "next_token": next_token.tolist()}
-            if rerun:
-                step["rerun_measured"] = True
-            if layer_probe:
-                step["layer_tokens"] = layer_tokens
-            trace.append(step)
-        if finished.all():
-            break
+    batch = model.begin_batch(len(prompt_tokens))
+    try:
+        for cur_pos in range(min(prompt_lens), total_len):
+            logits, info = model.step(tokens[:, prev_pos:cur_pos], prev_pos, batch, layer_probe=layer_probe)
+            next_token = (sample(logits, temperature) if temperature > 0 else logits.argmax(dim=-1)).view(-1)
+            next_token = torch.where(prompt_mask[:, cur_pos], tokens[:, cur_pos], next_token)
+            tokens[:, cur_pos] = next_token
+            finished |= torch.logical_and(~prompt_mask[:, cur_pos], next_token == eos_id)
+            prev_pos = cur_pos
+            if trace is not None:
+                trace.append({"pos": cur_pos, "next_token": next_token.tolist(), **info})
+            if finished.all():
+                break
+    finally:
+        model.end_batch(batch)
     completion_tokens = []
     for i, toks in enumerate(tokens.tolist()):
         toks = toks[prompt_lens[i]:prompt_lens[i] + max_new_tokens]
@@ -132,3 +112,43 @@ def generate(model, prompt_tokens: List[List[int]], max_new_tokens: int, eos_id:
             toks = toks[:toks.index(eos_id)]
         completion_tokens.append(toks)
     return completion_tokens
+
+
+def main(argv=None):
+    """Generates from prompts given as token ids (the checkpoints carry no tokenizer)."""
+    reg = _module("registry")
+    ap = argparse.ArgumentParser(prog="generate", description=main.__doc__)
+    ap.add_argument("--model", required=True, help="directory with config.json and *.safetensors (%s)"
+                    % ", ".join(reg.architectures()))
+    ap.add_argument("--tokens", action="append", default=[], metavar="IDS",
+                    help="one prompt: token ids separated by commas or spaces; may be given several times")
+    ap.add_argument("--input-file", help="JSON list of prompts, each a list of token ids")
+    ap.add_argument("--max-new-tokens", type=int, default=32)
+    ap.add_argument("--max-seq-len", type=int, default=4096)
+    ap.add_argument("--eos-id", type=int, default=-1)
+    ap.add_argument("--temperature", type=float, default=0.0)
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                    help="number format of the floating-point designs")
+    ap.add_argument("--layer-probe", action="store_true", help="report every layer's candidate token on stderr")
+    args = ap.parse_args(argv)
+    prompts = [[int(t) for t in p.replace(",", " ").split()] for p in args.tokens]
+    if args.input_file:
+        with open(args.input_file) as f:
+            prompts += json.load(f)
+    if not prompts or not all(prompts):
+        ap.error("give at least one prompt, none of them empty")
+    model = reg.load(args.model, dtype=args.dtype, max_seq_len=args.max_seq_len, max_batch_size=len(prompts))
+    vocab = model.args.vocab_size
+    if any(not 0 <= t < vocab for p in prompts for t in p):
+        ap.error("token ids go from 0 to %d" % (vocab - 1))
+    trace = [] if args.layer_probe else None
+    out = generate(model, prompts, args.max_new_tokens, args.eos_id, args.temperature, args.layer_probe, trace)
+    for step in trace or []:
+        print(json.dumps(step), file=sys.stderr)
+    for tokens in out:
+        print(json.dumps(tokens))
+    return 0
+
+
+if __name__ == "__main__":
+    sys.exit(main())

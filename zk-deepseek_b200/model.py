@@ -1002,6 +1002,53 @@ class Transformer(nn.Module):
         return logits
 
 
+    # -- the interface of generate.generate(), shared with the floating-point designs ------------------------
+    @property
+    def device(self):
+        return self.freqs_cis.device
+
+    def begin_batch(self, n):
+        """the caches hold the sequences of one batch, in order"""
+        return list(range(n))
+
+    def end_batch(self, batch):
+        pass
+
+    def _forward_step(self, toks, prev_pos, layer_probe):
+        """one pass over all layers; finish_inference raises ZkdsError if a kernel flagged its operands"""
+        h, start_pos, seqlen = self.prep_inference(toks, prev_pos)
+        layer_tokens = []
+        for i in range(self.args.n_layers):
+            h = self.layer_inference(i, h, start_pos, seqlen)
+            if layer_probe:
+                probe = self.head(self.norm(h)[0][:, -1].contiguous()[None, :])
+                layer_tokens.append(probe.argmax(dim=-1).view(-1).tolist())
+        return self.finish_inference(h), layer_tokens
+
+    @torch.inference_mode()
+    def step(self, toks, prev_pos, batch=None, layer_probe=False):
+        """(logits of the last position, info): runs toks [B, S] of sequences that stand at prev_pos, writes the
+        step's tokens.bin under `snark`"""
+        if snark:
+            os.makedirs(f"{zkDataDir}/pos_{prev_pos}", exist_ok=True)
+            saveTensor(f"{zkDataDir}/pos_{prev_pos}/tokens.bin", toks[0].cpu())
+        info = {}
+        try:
+            logits, layer_tokens = self._forward_step(toks, prev_pos, layer_probe)
+        except K.ZkdsError as err:
+            if err.status != K.ERR_RANGE:
+                raise
+            # an activation exceeded the limb bound promised for it (ACT_LIMBS, MLA.score_limbs): that pass's
+            # numbers are wrong.  The step only wrote cache rows it owns, so it is simply run again with every
+            # limb count measured on the device.
+            with measured_limbs(self):
+                logits, layer_tokens = self._forward_step(toks, prev_pos, layer_probe)
+            info["rerun_measured"] = True
+        if layer_probe:
+            info["layer_tokens"] = layer_tokens
+        return logits, info
+
+
 class measured_limbs:
     """Context manager: every activation's limb count is measured on the device (ACT_LIMBS = 0, score
     contractions included) instead of promised.  Slower (one host synchronisation per GEMM), never wrong;
