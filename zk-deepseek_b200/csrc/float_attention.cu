@@ -1,8 +1,368 @@
+// Windowed softmax attention on the tensor cores, bfloat16 operands, 32-bit scores, weights and sums.
+//
+// attention_expanded_kernel (prefill): per-head keys [k1 | k2] and values.  A CTA owns one head and two tiles of 128
+// query tokens; keys come in tiles of 128.  Tensor memory holds both score tiles and both output tiles; the bfloat16
+// weights overwrite the scores they came from and feed the second product from tensor memory.  While one query tile is
+// in its softmax the tensor core works for the other.
+//   warp 0      TMA loads          warp 1      MMA issue
+//   warps 2-5   softmax, tile 0    warps 6-9   softmax, tile 1 (one query row per thread)
+// The running maximum only replaces the one in use when it has grown by more than 2^8; the output tile is then
+// rescaled in place.  A commit covers every MMA issued before it, so "scores ready" also says that the output tile is
+// free to be rescaled.
+#include <cuda.h>
+
 #include "float_common.cuh"
+#include "tcgen05.cuh"
+
 namespace zkds {
-bool attention_prefill_tc_takes(const zkfp_attention_args&) { return false; }
-int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st) { return launch_attention_plain(a, st); }
+
+bool fp_tensor_map(CUtensorMap* map, const void* base, int rank, const uint64_t* dims, const uint64_t* strides_bytes,
+                   const uint32_t* box);
+
+namespace {
+
+constexpr int kTile = 128;                     // query rows and keys per tile
+constexpr uint32_t kSeg = kTile * 128;         // bytes of 128 rows x 64 bfloat16
+constexpr int kThreadsAttn = 320;
+constexpr size_t kSmemMax = 226 * 1024;
+
+__device__ __forceinline__ float exp2_approx(float x)
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+struct ExpandedParams {
+    bf16* out;
+    const int* start;
+    long long o_head;
+    int seq, heads, base, window;
+    int d1, d2, dv, seg1, seg2, segv;          // segments of 64 columns
+    int k_stages, v_stages;
+    float scale_log2;                          // scale * log2(e)
+    int* error_flag;
+};
+
+struct ExpandedShared {
+    uint64_t q_full, k_full[4], k_empty[4], v_full[4], v_empty[4], s_full[2], p_full[2], o_full[2];
+    uint32_t tmem;
+    int abort;
+};
+
+// key tiles of one block of query tiles: tile j covers positions lo + 128 j ..; tile g is active for first[g] .. last[g]
+struct KeyTiles {
+    int lo, n, first[2], last[2];
+};
+
+__device__ __forceinline__ KeyTiles key_tiles(const ExpandedParams& p, int t0, int start)
+{
+    KeyTiles k;
+    const int lo0 = p.window > 0 ? start + t0 - p.window + 1 : 0;
+    k.lo = lo0 > p.base ? lo0 : p.base;
+    k.n = 0;
+#pragma unroll
+    for (int g = 0; g < 2; ++g) {
+        const int r0 = t0 + g * kTile;
+        if (r0 >= p.seq) { k.first[g] = 1; k.last[g] = 0; continue; }
+        const int r1 = min(r0 + kTile, p.seq) - 1;
+        const int lo = p.window > 0 ? max(start + r0 - p.window + 1, k.lo) : k.lo;
+        k.first[g] = (lo - k.lo) / kTile;
+        k.last[g] = (start + r1 - k.lo) / kTile;
+        k.n = max(k.n, k.last[g] + 1);
+    }
+    return k;
+}
+
+__global__ void __launch_bounds__(kThreadsAttn, 1)
+attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid_constant__ CUtensorMap tmQ2,
+                          const __grid_constant__ CUtensorMap tmK1, const __grid_constant__ CUtensorMap tmK2,
+                          const __grid_constant__ CUtensorMap tmV, const ExpandedParams p)
+{
+    extern __shared__ uint8_t raw[];
+    uint8_t* base = (uint8_t*)(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
+    __shared__ ExpandedShared s;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.y, t0 = (int)(gridDim.x - 1 - blockIdx.x) * 2 * kTile;    // longest blocks first
+    const int start = p.start[0];
+    const KeyTiles kt = key_tiles(p, t0, start);
+    const int segq = p.seg1 + p.seg2;
+    const uint32_t sQ = smem_u32(base), bytesQ = (uint32_t)segq * kSeg;
+    const uint32_t sK = sQ + 2 * bytesQ, sV = sK + (uint32_t)p.k_stages * bytesQ, bytesV = (uint32_t)p.segv * kSeg;
+    volatile int* abort_flag = &s.abort;
+
+    if (threadIdx.x == 0) {
+        s.abort = 0;
+        mbar_init(smem_u32(&s.q_full), 1);
+        for (int i = 0; i < 4; ++i) {
+            mbar_init(smem_u32(&s.k_full[i]), 1);
+            mbar_init(smem_u32(&s.k_empty[i]), 1);
+            mbar_init(smem_u32(&s.v_full[i]), 1);
+            mbar_init(smem_u32(&s.v_empty[i]), 1);
+        }
+        for (int g = 0; g < 2; ++g) {
+            mbar_init(smem_u32(&s.s_full[g]), 1);
+            mbar_init(smem_u32(&s.p_full[g]), 4);
+            mbar_init(smem_u32(&s.o_full[g]), 1);
+        }
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncwarp();
+    if (warp == 1) tmem_alloc(smem_u32(&s.tmem), 512);
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s.tmem;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            const int tiles_q = t0 + kTile < p.seq ? 2 : 1;
+            mbar_expect_tx(smem_u32(&s.q_full), (uint32_t)tiles_q * bytesQ);
+            for (int g = 0; g < tiles_q; ++g) {
+                for (int c = 0; c < p.seg1; ++c)
+                    tma_load_3d(sQ + g * bytesQ + c * kSeg, &tmQ1, c * 64, head, t0 + g * kTile, smem_u32(&s.q_full));
+                for (int c = 0; c < p.seg2; ++c)
+                    tma_load_3d(sQ + g * bytesQ + (p.seg1 + c) * kSeg, &tmQ2, c * 64, head, t0 + g * kTile,
+                                smem_u32(&s.q_full));
+            }
+            int ks = 0, vs = 0;
+            uint32_t kp = 0, vp = 0;
+            for (int j = 0; j < kt.n; ++j) {
+                const int y = kt.lo - p.base + j * kTile;
+                if (!mbar_wait(smem_u32(&s.k_empty[ks]), kp ^ 1u, abort_flag)) break;
+                uint32_t bar = smem_u32(&s.k_full[ks]), dst = sK + (uint32_t)ks * bytesQ;
+                mbar_expect_tx(bar, bytesQ);
+                for (int c = 0; c < p.seg1; ++c) tma_load_3d(dst + c * kSeg, &tmK1, c * 64, head, y, bar);
+                for (int c = 0; c < p.seg2; ++c) tma_load_2d(dst + (p.seg1 + c) * kSeg, &tmK2, c * 64, y, bar);
+                if (++ks == p.k_stages) { ks = 0; kp ^= 1u; }
+                if (!mbar_wait(smem_u32(&s.v_empty[vs]), vp ^ 1u, abort_flag)) break;
+                bar = smem_u32(&s.v_full[vs]);
+                dst = sV + (uint32_t)vs * bytesV;
+                mbar_expect_tx(bar, bytesV);
+                for (int c = 0; c < p.segv; ++c) tma_load_3d(dst + c * kSeg, &tmV, c * 64, head, y, bar);
+                if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc_s = idesc_bf16(kTile, kTile), idesc_o = idesc_bf16(kTile, (p.dv + 15) & ~15, true);
+            const int steps1 = (p.d1 + 15) / 16, steps2 = (p.d2 + 15) / 16;
+            uint32_t pp[2] = {0, 0};
+            int ks = 0, vs = 0;
+            uint32_t kp = 0, vp = 0;
+            auto scores = [&](int g) {
+                const uint32_t a = sQ + (uint32_t)g * bytesQ, b = sK + (uint32_t)ks * bytesQ, d = tmem + (uint32_t)g * kTile;
+                uint32_t acc = 0;
+                for (int k = 0; k < steps1 + steps2; ++k) {
+                    const int kk = k < steps1 ? k : p.seg1 * 4 + (k - steps1);       // 16-column step inside the tile
+                    const uint32_t off = (uint32_t)(kk >> 2) * kSeg + (uint32_t)(kk & 3) * 32u;
+                    umma_bf16(d, smem_desc_sw128(a + off), smem_desc_sw128(b + off), idesc_s, acc);
+                    acc = 1;
+                }
+                umma_commit(smem_u32(&s.s_full[g]));
+            };
+            auto active = [&](int g, int j) { return j >= kt.first[g] && j <= kt.last[g]; };
+            bool ok = mbar_wait(smem_u32(&s.q_full), 0, abort_flag);
+            for (int j = -1; j < kt.n && ok; ++j) {
+                if (j >= 0 && !(ok = mbar_wait(smem_u32(&s.v_full[vs]), vp, abort_flag))) break;
+                const bool next = j + 1 < kt.n;
+                bool k_ready = false;
+                for (int g = 0; g < 2 && ok; ++g) {
+                    if (j >= 0 && active(g, j)) {
+                        if (!(ok = mbar_wait(smem_u32(&s.p_full[g]), pp[g], abort_flag))) break;
+                        pp[g] ^= 1u;
+                        tc_fence_after();
+                        const uint32_t a = tmem + (uint32_t)g * kTile, d = tmem + 256u + (uint32_t)g * kTile;
+#pragma unroll
+                        for (int k = 0; k < kTile / 16; ++k)
+                            umma_bf16_ts(d, a + (uint32_t)k * 8u,
+                                         smem_desc_mn_sw128(sV + (uint32_t)vs * bytesV + (uint32_t)k * 2048u, kSeg), idesc_o,
+                                         (j > kt.first[g] || k) ? 1u : 0u);
+                        if (j == kt.last[g]) umma_commit(smem_u32(&s.o_full[g]));
+                    }
+                    if (next && active(g, j + 1)) {
+                        if (!k_ready) {
+                            if (!(ok = mbar_wait(smem_u32(&s.k_full[ks]), kp, abort_flag))) break;
+                            tc_fence_after();
+                            k_ready = true;
+                        }
+                        scores(g);
+                    }
+                }
+                // a stage is handed back only after its load has landed, also when no query tile used it
+                if (ok && next && !k_ready) ok = mbar_wait(smem_u32(&s.k_full[ks]), kp, abort_flag);
+                if (!ok) break;
+                if (j >= 0) {
+                    umma_commit(smem_u32(&s.v_empty[vs]));
+                    if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }
+                }
+                if (next) {
+                    umma_commit(smem_u32(&s.k_empty[ks]));
+                    if (++ks == p.k_stages) { ks = 0; kp ^= 1u; }
+                }
+            }
+        }
+    } else {
+        const int g = (warp - 2) >> 2, quarter = warp & 3, row = quarter * 32 + lane;
+        const int t = t0 + g * kTile + row, pos = start + t;
+        const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
+        const uint32_t tS = tmem + (uint32_t)g * kTile + lanes, tO = tmem + 256u + (uint32_t)g * kTile + lanes;
+        float m_used = -INFINITY, l = 0.f;
+        uint32_t sp = 0;
+        bool ok = true;
+        for (int j = kt.first[g]; j <= kt.last[g]; ++j) {
+            if (!(ok = mbar_wait(smem_u32(&s.s_full[g]), sp, abort_flag))) break;
+            sp ^= 1u;
+            tc_fence_after();
+            // visible columns of this row: c_lo .. c_hi
+            const int j0 = kt.lo + j * kTile;
+            const int c_hi = pos - j0, c_lo = p.window > 0 ? c_hi - p.window + 1 : -1;
+            const bool masked = __any_sync(0xffffffffu, c_hi < kTile - 1 || c_lo > 0);
+            float mx = -INFINITY;
+#pragma unroll
+            for (int c = 0; c < kTile; c += 32) {
+                float v[32];
+                tmem_ld32(tS + (uint32_t)c, v);
+                tmem_ld_wait();
+                if (masked) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if (c + i >= c_lo && c + i <= c_hi) mx = fmaxf(mx, v[i]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, v[i]);
+                }
+            }
+            const float m_new = fmaxf(m_used, mx * p.scale_log2);
+            if (j == kt.first[g]) {
+                m_used = m_new;
+            } else if (__any_sync(0xffffffffu, m_new > m_used + 8.0f)) {
+                const float f = m_used == -INFINITY ? 0.f : exp2_approx(m_used - m_new);
+                for (int c = 0; c < p.dv; c += 32) {
+                    float v[32];
+                    tmem_ld32(tO + (uint32_t)c, v);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] *= f;
+                    tmem_st32(tO + (uint32_t)c, v);
+                }
+                l *= f;
+                m_used = m_new;
+            }
+            const float m_sub = m_used == -INFINITY ? 0.f : m_used;
+#pragma unroll
+            for (int c = 0; c < kTile; c += 32) {
+                float v[32];
+                tmem_ld32(tS + (uint32_t)c, v);
+                tmem_ld_wait();
+                uint32_t w[16];
+#pragma unroll
+                for (int i = 0; i < 32; ++i) v[i] = exp2_approx(fmaf(v[i], p.scale_log2, -m_sub));
+                if (masked) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if (c + i < c_lo || c + i > c_hi) v[i] = 0.f;
+                }
+                float part = 0.f;
+#pragma unroll
+                for (int i = 0; i < 32; ++i) part += v[i];
+                l += part;
+#pragma unroll
+                for (int i = 0; i < 16; ++i) w[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
+                tmem_st16(tS + (uint32_t)(c / 2), w);
+            }
+            tmem_st_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&s.p_full[g]));
+        }
+        if (ok && kt.first[g] <= kt.last[g] && mbar_wait(smem_u32(&s.o_full[g]), 0, abort_flag)) {
+            tc_fence_after();
+            const float r = 1.0f / l;
+            bf16* o = p.out + ((long long)t * p.heads + head) * p.o_head;
+            for (int c = 0; c < p.dv; c += 32) {
+                float v[32];
+                tmem_ld32(tO + (uint32_t)c, v);
+                tmem_ld_wait();
+                if (t < p.seq) {
+#pragma unroll
+                    for (int i = 0; i < 32; i += 8) {
+                        if (c + i < p.dv) {
+                            float w[8];
+#pragma unroll
+                            for (int k = 0; k < 8; ++k) w[k] = v[i + k] * r;
+                            store8(o + c + i, w);
+                        }
+                    }
+                }
+            }
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 1) tmem_dealloc(tmem, 512);
+    if (threadIdx.x == 0 && s.abort) *(volatile int*)p.error_flag = 1;
+}
+
+size_t expanded_smem(const zkfp_attention_args& a, int& ks, int& vs)
+{
+    const size_t segq = (size_t)(a.d1 + 63) / 64 + (a.d2 + 63) / 64, segv = (a.dv + 63) / 64;
+    ks = vs = 1;
+    auto bytes = [&] { return 1024 + kSeg * ((2 + ks) * segq + vs * segv); };
+    if (bytes() > kSmemMax) return 0;
+    ++ks;
+    if (bytes() > kSmemMax) { --ks; return bytes(); }
+    ++vs;
+    if (bytes() > kSmemMax) --vs;
+    return bytes();
+}
+
+}  // namespace
+
+bool attention_prefill_tc_takes(const zkfp_attention_args& a)
+{
+    int ks, vs;
+    return a.dtype == ZKFP_BF16 && !a.shared && a.batch == 1 && a.dv <= 128 && a.keys > 0 &&
+           a.keys < 0x40000000 && a.seq < 0x40000000 && expanded_smem(a, ks, vs) > 0 &&
+           !((a.q_head | a.k1_tok | a.k1_head | a.k2_tok | a.v_tok | a.v_head | a.o_head) & 7) &&
+           !(((uintptr_t)a.q | (uintptr_t)a.k1 | (uintptr_t)a.k2 | (uintptr_t)a.v | (uintptr_t)a.out) & 15);
+}
+
+int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st)
+{
+    ExpandedParams p;
+    p.out = (bf16*)a.out; p.start = a.start; p.o_head = a.o_head;
+    p.seq = (int)a.seq; p.heads = (int)a.heads; p.base = (int)a.base; p.window = a.window;
+    p.d1 = a.d1; p.d2 = a.d2; p.dv = a.dv;
+    p.seg1 = (a.d1 + 63) / 64; p.seg2 = (a.d2 + 63) / 64; p.segv = (a.dv + 63) / 64;
+    p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.error_flag = fp_error_flag();
+    if (!p.error_flag) return ZKDS_ERR_WORKSPACE;
+    const size_t smem = expanded_smem(a, p.k_stages, p.v_stages);
+    CUtensorMap q1, q2, k1, k2, v;
+    const uint64_t H = (uint64_t)a.heads, S = (uint64_t)a.seq, N = (uint64_t)a.keys;
+    const uint64_t qs[2] = {(uint64_t)a.q_head * 2, (uint64_t)a.q_head * 2 * H};
+    const uint64_t ks[2] = {(uint64_t)a.k1_head * 2, (uint64_t)a.k1_tok * 2}, k2s[1] = {(uint64_t)a.k2_tok * 2};
+    const uint64_t vs[2] = {(uint64_t)a.v_head * 2, (uint64_t)a.v_tok * 2};
+    const uint64_t dq1[3] = {(uint64_t)a.d1, H, S}, dq2[3] = {(uint64_t)(a.d2 ? a.d2 : 8), H, S};
+    const uint64_t dk1[3] = {(uint64_t)a.d1, H, N}, dk2[2] = {(uint64_t)(a.d2 ? a.d2 : 8), N}, dv[3] = {(uint64_t)a.dv, H, N};
+    const uint32_t b3[3] = {64, 1, kTile}, b2[2] = {64, kTile};
+    const bf16* q = (const bf16*)a.q;
+    if (!fp_tensor_map(&q1, q, 3, dq1, qs, b3) || !fp_tensor_map(&q2, a.d2 ? q + a.d1 : q, 3, dq2, qs, b3) ||
+        !fp_tensor_map(&k1, a.k1, 3, dk1, ks, b3) || !fp_tensor_map(&k2, a.k2, 2, dk2, k2s, b2) ||
+        !fp_tensor_map(&v, a.v, 3, dv, vs, b3))
+        return ZKDS_ERR_UNSUPPORTED;
+    ZKDS_CUDA(cudaFuncSetAttribute(attention_expanded_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
+    // more than half the shared memory: one CTA per SM, so the tensor-memory allocation never waits
+    const size_t want = smem < 120 * 1024 ? 120 * 1024 : smem;
+    const dim3 grid((unsigned)((a.seq + 2 * kTile - 1) / (2 * kTile)), (unsigned)a.heads);
+    attention_expanded_kernel<<<grid, kThreadsAttn, want, st>>>(q1, q2, k1, k2, v, p);
+    return fp_launched();
+}
+
 bool attention_decode_tc_takes(const zkfp_attention_args&) { return false; }
 int launch_attention_decode_tc(const zkfp_attention_args& a, cudaStream_t st) { return launch_attention_plain(a, st); }
 long long attention_decode_scratch(const zkfp_attention_args&) { return 0; }
-}
+
+}  // namespace zkds
