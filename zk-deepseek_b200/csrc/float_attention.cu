@@ -361,8 +361,279 @@ int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st)
     return fp_launched();
 }
 
-bool attention_decode_tc_takes(const zkfp_attention_args&) { return false; }
-int launch_attention_decode_tc(const zkfp_attention_args& a, cudaStream_t st) { return launch_attention_plain(a, st); }
-long long attention_decode_scratch(const zkfp_attention_args&) { return 0; }
+// ---- attention over the latents (decode) -------------------------------------------------------------------------
+// Rows are (token, head) pairs, all heads read the same keys, and the values are the latent part of the keys.  A CTA
+// takes 128 rows and one chunk of 64 keys: scores, softmax of the chunk, weighted sum; partial results go to scratch
+// and latent_combine_kernel merges the chunks.  The key tile in shared memory serves both products (keys x latent as
+// the K-major operand of the scores and as the N-major operand of the sum), so the cache is read once.  The
+// weights take the place of the queries in shared memory and the sums that of the scores in tensor memory.
+namespace {
+
+constexpr int kChunk = 64;
+constexpr uint32_t kSegC = kChunk * 128;       // bytes of 64 keys x 64 columns
+
+struct LatentParams {
+    const int* start;
+    const int* slots;
+    float* part;               // [batch][row tile][chunk][c][128]
+    float* ml;                 // [batch][row tile][chunk][2][128]: maximum (log2 units), sum
+    int rows, heads, seq, window, c, r, segc, segr, chunks, row_tiles;
+    float scale_log2;
+    int* error_flag;
+};
+
+struct LatentShared {
+    uint64_t q_full, k_full, s_full, p_full, o_full;
+    uint32_t tmem;
+    int abort;
+};
+
+// first chunk (in units of kChunk positions) and number of chunks of a row tile
+__device__ __forceinline__ void chunk_range(int start, int row0, int rows, int heads, int window, int& first, int& n)
+{
+    const int last_row = min(row0 + kTile, rows) - 1;
+    const int lo = window > 0 ? max(start + row0 / heads - window + 1, 0) : 0;
+    const int hi = start + last_row / heads;
+    first = lo / kChunk;
+    n = hi / kChunk - first + 1;
+}
+
+__global__ void __launch_bounds__(192, 1)
+attention_latent_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid_constant__ CUtensorMap tmQ2,
+                        const __grid_constant__ CUtensorMap tmK1, const __grid_constant__ CUtensorMap tmK2,
+                        const LatentParams p)
+{
+    extern __shared__ uint8_t raw[];
+    __shared__ LatentShared s;
+    const int b = blockIdx.z, row0 = blockIdx.y * kTile, start = p.start[b];
+    int first, n;
+    chunk_range(start, row0, p.rows, p.heads, p.window, first, n);
+    if ((int)blockIdx.x >= n) return;
+    const int j0 = (first + (int)blockIdx.x) * kChunk;
+    uint8_t* base = (uint8_t*)(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, seg = p.segc + p.segr;
+    const uint32_t sQ = smem_u32(base), sK = sQ + (uint32_t)seg * kSeg;
+    volatile int* abort_flag = &s.abort;
+    if (threadIdx.x == 0) {
+        s.abort = 0;
+        mbar_init(smem_u32(&s.q_full), 1);
+        mbar_init(smem_u32(&s.k_full), 1);
+        mbar_init(smem_u32(&s.s_full), 1);
+        mbar_init(smem_u32(&s.p_full), 4);
+        mbar_init(smem_u32(&s.o_full), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncwarp();
+    if (warp == 1) tmem_alloc(smem_u32(&s.tmem), 512);
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s.tmem;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            const uint32_t kb = smem_u32(&s.k_full), qb = smem_u32(&s.q_full);
+            const int y = b * p.rows + row0, slot = p.slots ? p.slots[b] : b;
+            mbar_expect_tx(kb, (uint32_t)seg * kSegC);
+            mbar_expect_tx(qb, (uint32_t)seg * kSeg);
+            for (int c = 0; c < seg; ++c) {
+                const bool lat = c < p.segc;
+                const int x = (lat ? c : c - p.segc) * 64;
+                tma_load_3d(sK + (uint32_t)c * kSegC, lat ? &tmK1 : &tmK2, x, j0, slot, kb);
+                tma_load_2d(sQ + (uint32_t)c * kSeg, lat ? &tmQ1 : &tmQ2, x, y, qb);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            bool ok = mbar_wait(smem_u32(&s.q_full), 0, abort_flag) && mbar_wait(smem_u32(&s.k_full), 0, abort_flag);
+            if (ok) {
+                tc_fence_after();
+                const uint32_t idesc = idesc_bf16(kTile, kChunk);
+                const int steps1 = (p.c + 15) / 16, steps2 = (p.r + 15) / 16;
+                for (int k = 0; k < steps1 + steps2; ++k) {
+                    const int kk = k < steps1 ? k : p.segc * 4 + (k - steps1);
+                    umma_bf16(tmem, smem_desc_sw128(sQ + (uint32_t)(kk >> 2) * kSeg + (uint32_t)(kk & 3) * 32u),
+                              smem_desc_sw128(sK + (uint32_t)(kk >> 2) * kSegC + (uint32_t)(kk & 3) * 32u), idesc,
+                              k ? 1u : 0u);
+                }
+                umma_commit(smem_u32(&s.s_full));
+                ok = mbar_wait(smem_u32(&s.p_full), 0, abort_flag);
+            }
+            if (ok) {
+                tc_fence_after();
+                for (int n0 = 0; n0 < p.c; n0 += 256) {
+                    const int w = (min(p.c - n0, 256) + 15) & ~15;
+                    const uint32_t idesc = idesc_bf16(kTile, w, true);
+#pragma unroll
+                    for (int k = 0; k < kChunk / 16; ++k)
+                        umma_bf16(tmem + (uint32_t)n0, smem_desc_sw128(sQ + (uint32_t)k * 32u),
+                                  smem_desc_mn_sw128(sK + (uint32_t)(n0 / 64) * kSegC + (uint32_t)k * 2048u, kSegC), idesc,
+                                  k ? 1u : 0u);
+                }
+                umma_commit(smem_u32(&s.o_full));
+            }
+        }
+    } else {
+        const int quarter = warp & 3, row = quarter * 32 + lane, rr = row0 + row;
+        const uint32_t tq = tmem + ((uint32_t)(quarter * 32) << 16);
+        const bool row_ok = rr < p.rows;
+        const int c_hi = start + rr / p.heads - j0, c_lo = p.window > 0 ? c_hi - p.window + 1 : 0;
+        const long long tile = ((long long)b * p.row_tiles + blockIdx.y) * p.chunks + blockIdx.x;
+        if (mbar_wait(smem_u32(&s.s_full), 0, abort_flag)) {
+            tc_fence_after();
+            float v[2][32];
+            tmem_ld32(tq, v[0]);
+            tmem_ld32(tq + 32u, v[1]);
+            tmem_ld_wait();
+            float m = -INFINITY, l = 0.f;
+#pragma unroll
+            for (int i = 0; i < 64; ++i) {
+                float& x = v[i >> 5][i & 31];
+                x = row_ok && i >= c_lo && i <= c_hi ? x * p.scale_log2 : -INFINITY;
+                m = fmaxf(m, x);
+            }
+            const float m_sub = m == -INFINITY ? 0.f : m;
+#pragma unroll
+            for (int i = 0; i < 64; ++i) {
+                float& x = v[i >> 5][i & 31];
+                x = exp2_approx(x - m_sub);
+                l += x;
+            }
+            // 128 bytes of bfloat16 weights per row, 16-byte pieces swizzled as TMA would have written them
+            uint8_t* dst = base + row * 128;
+#pragma unroll
+            for (int q = 0; q < 8; ++q) {
+                const float* x = &v[q >> 2][(q & 3) * 8];
+                *reinterpret_cast<uint4*>(dst + ((q ^ (row & 7)) << 4)) =
+                    make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&s.p_full));
+            if (row_ok) {
+                p.ml[tile * 256 + row] = m;
+                p.ml[tile * 256 + 128 + row] = l;
+            }
+            if (mbar_wait(smem_u32(&s.o_full), 0, abort_flag)) {
+                tc_fence_after();
+                float* out = p.part + tile * p.c * 128 + row;
+                for (int c = 0; c < p.c; c += 32) {
+                    tmem_ld32(tq + (uint32_t)c, v[0]);
+                    tmem_ld_wait();
+                    if (row_ok) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                            if (c + i < p.c) out[(long long)(c + i) * 128] = v[0][i];
+                    }
+                }
+            }
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 1) tmem_dealloc(tmem, 512);
+    if (threadIdx.x == 0 && s.abort) *(volatile int*)p.error_flag = 1;
+}
+
+// merges the chunks of 32 rows x 32 latent columns.  grid (c / 32, row tiles * 4, batch)
+__global__ void __launch_bounds__(256)
+latent_combine_kernel(const LatentParams p, bf16* __restrict__ out, long long o_head)
+{
+    __shared__ float tile[32][33];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.z;
+    const int rt = blockIdx.y >> 2, row = (blockIdx.y & 3) * 32 + lane, row0 = rt * kTile, c0 = blockIdx.x * 32;
+    if (row0 + (int)(blockIdx.y & 3) * 32 >= p.rows) return;
+    int first, n;
+    chunk_range(p.start[b], row0, p.rows, p.heads, p.window, first, n);
+    const long long t0 = ((long long)b * p.row_tiles + rt) * p.chunks;
+    const float* ml = p.ml + t0 * 256 + row;
+    const bool row_ok = row0 + row < p.rows;
+    float m = -INFINITY;
+    if (row_ok)
+#pragma unroll 8
+        for (int i = 0; i < n; ++i) m = fmaxf(m, ml[(long long)i * 256]);
+    float acc[4] = {}, l = 0.f;
+    const int c = c0 + warp * 4;
+    if (row_ok && c < p.c) {
+        const float* src = p.part + (t0 * p.c + c) * 128 + row;
+#pragma unroll 4
+        for (int i = 0; i < n; ++i) {
+            const float w = exp2_approx(ml[(long long)i * 256] - m);
+            l = fmaf(w, ml[(long long)i * 256 + 128], l);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) acc[k] = fmaf(w, src[((long long)i * p.c + k) * 128], acc[k]);
+        }
+    }
+    const float r = 1.0f / l;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) tile[warp * 4 + k][lane] = acc[k] * r;
+    __syncthreads();
+    for (int i = warp; i < 32; i += 8) {
+        const int rr = row0 + (int)(blockIdx.y & 3) * 32 + i;
+        if (rr < p.rows && c0 + lane < p.c)
+            out[((long long)b * p.rows + rr) * o_head + c0 + lane] = __float2bfloat16_rn(tile[lane][i]);
+    }
+}
+
+int latent_chunks(const zkfp_attention_args& a) { return (a.max_keys + kChunk - 1) / kChunk + 1; }
+
+size_t latent_smem(const zkfp_attention_args& a)
+{
+    return 1024 + (size_t)((a.d1 + 63) / 64 + (a.d2 + 63) / 64) * (kSeg + kSegC);
+}
+
+}  // namespace
+
+bool attention_decode_tc_takes(const zkfp_attention_args& a)
+{
+    return a.dtype == ZKFP_BF16 && a.shared && a.v == a.k1 && a.dv == a.d1 && a.v_tok == a.k1_tok && a.d1 <= 512 &&
+           a.k2_tok == a.k1_tok && a.base == 0 && a.keys > 0 && a.max_keys > 0 && latent_smem(a) <= kSmemMax &&
+           a.seq * a.heads < 0x1000000 && !((a.q_head | a.k1_tok | a.o_head | a.slot_stride) & 7) &&
+           !(((uintptr_t)a.q | (uintptr_t)a.k1 | (uintptr_t)a.k2 | (uintptr_t)a.out) & 15);
+}
+
+long long attention_decode_scratch(const zkfp_attention_args& a)
+{
+    const long long row_tiles = (a.seq * a.heads + kTile - 1) / kTile;
+    return a.batch * row_tiles * latent_chunks(a) * 128 * (a.d1 + 2);
+}
+
+int launch_attention_decode_tc(const zkfp_attention_args& a, cudaStream_t st)
+{
+    if (!a.scratch) return ZKDS_ERR_ARG;
+    LatentParams p;
+    p.start = a.start; p.slots = a.slots;
+    p.rows = (int)(a.seq * a.heads); p.heads = (int)a.heads; p.seq = (int)a.seq; p.window = a.window;
+    p.c = a.d1; p.r = a.d2; p.segc = (a.d1 + 63) / 64; p.segr = (a.d2 + 63) / 64;
+    p.chunks = latent_chunks(a);
+    p.row_tiles = (p.rows + kTile - 1) / kTile;
+    p.part = a.scratch;
+    p.ml = a.scratch + (long long)a.batch * p.row_tiles * p.chunks * 128 * p.c;
+    p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.error_flag = fp_error_flag();
+    if (!p.error_flag) return ZKDS_ERR_WORKSPACE;
+    CUtensorMap q1, q2, k1, k2;
+    const uint64_t rows = (uint64_t)(a.batch * p.rows), r = (uint64_t)(a.d2 ? a.d2 : 8);
+    const uint64_t dq1[2] = {(uint64_t)a.d1, rows}, dq2[2] = {r, rows}, qs[1] = {(uint64_t)a.q_head * 2};
+    // the slot extent only bounds the coordinate; slots are valid by construction
+    const uint64_t dk1[3] = {(uint64_t)a.d1, (uint64_t)a.keys, 65536}, dk2[3] = {r, (uint64_t)a.keys, 65536};
+    const uint64_t ks[2] = {(uint64_t)a.k1_tok * 2, (uint64_t)a.slot_stride * 2};
+    const uint32_t bq[2] = {64, kTile}, bk[3] = {64, kChunk, 1};
+    const bf16* q = (const bf16*)a.q;
+    if (!fp_tensor_map(&q1, q, 2, dq1, qs, bq) || !fp_tensor_map(&q2, a.d2 ? q + a.d1 : q, 2, dq2, qs, bq) ||
+        !fp_tensor_map(&k1, a.k1, 3, dk1, ks, bk) || !fp_tensor_map(&k2, a.d2 ? a.k2 : a.k1, 3, dk2, ks, bk))
+        return ZKDS_ERR_UNSUPPORTED;
+    ZKDS_CUDA(cudaFuncSetAttribute(attention_latent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
+    const size_t smem = latent_smem(a) < 120 * 1024 ? 120 * 1024 : latent_smem(a);
+    attention_latent_kernel<<<dim3((unsigned)p.chunks, (unsigned)p.row_tiles, (unsigned)a.batch), 192, smem, st>>>(q1, q2, k1,
+                                                                                                             k2, p);
+    int rc = fp_launched();
+    if (rc != ZKDS_OK) return rc;
+    latent_combine_kernel<<<dim3((unsigned)((p.c + 31) / 32), (unsigned)p.row_tiles * 4, (unsigned)a.batch), 256, 0, st>>>(
+        p, (bf16*)a.out, a.o_head);
+    return fp_launched();
+}
 
 }  // namespace zkds
