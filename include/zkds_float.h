@@ -30,7 +30,7 @@ typedef struct {
     const float* table;    /* rotate: (cos, sin) pairs, [position][pairs] */
     const int* start;      /* rotate: first position of every sequence */
     long long lda, ldw, ldo, ldaux;
-    long long M, N, K;     /* N, K padded */
+    long long M, N, K;     /* N, K padded (GLU: N a multiple of 16) */
     long long seq;         /* rotate: rows per sequence */
     int dtype, out_dtype, epilogue;
     int pairs, period, offset;

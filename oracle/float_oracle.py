@@ -1,10 +1,17 @@
 """Plain, slow restatement of the floating-point decoder designs: numpy in float64, one function per
 mechanism, one sequence at a time, no cache.  Test infrastructure; it shares no code with the product path.
 
+`rnd` is applied to every activation that a reduced-precision run stores between its products (identity by default):
+with a rounding function the result shows the error that rounding alone causes.
+
 A sequence is an array of token ids; activations are [tokens, width].  `W` maps tensor names to arrays and
 `cfg` is the parsed configuration.  Linear weights are [out, in].
 """
 import numpy as np
+
+
+def exact(x):
+    return x
 
 
 def rms_norm(x, w, eps):
@@ -45,42 +52,43 @@ def softmax_rows(s, visible):
     return e / e.sum(axis=-1, keepdims=True)
 
 
-def latent_kv(h, W, p, mx, eps):
+def latent_kv(h, W, p, mx, eps, rnd=exact):
     """the two cached parts of every token: the normed latent [T, C] and the rotated shared key part [T, R]"""
     y = h @ W[p + "dkv"].T
     C = mx["kv_rank"]
     c = rms_norm(y[:, :C], W[p + "dkv.norm"], eps)
-    return c, rotate_pairs(y[:, C:], np.arange(len(h), dtype=np.float64), mx["rot"]["base"])
+    return rnd(c), rnd(rotate_pairs(y[:, C:], np.arange(len(h), dtype=np.float64), mx["rot"]["base"]))
 
 
-def latent_queries(h, W, p, mx, eps):
+def latent_queries(h, W, p, mx, eps, rnd=exact):
     """per head the unrotated [T, H, D] and the rotated [T, H, R] query"""
     H, D, R = mx["heads"], mx["dim"], mx["rot_dim"]
-    cq = rms_norm(h @ W[p + "dq"].T, W[p + "dq.norm"], eps)
+    cq = rnd(rms_norm(h @ W[p + "dq"].T, W[p + "dq.norm"], eps))
     q = (cq @ W[p + "uq"].T).reshape(len(h), H, D + R)
-    return q[:, :, :D], rotate_pairs(q[:, :, D:], np.arange(len(h), dtype=np.float64), mx["rot"]["base"])
+    turned = rotate_pairs(q[:, :, D:], np.arange(len(h), dtype=np.float64), mx["rot"]["base"])
+    return rnd(q[:, :, :D]), rnd(turned)
 
 
-def latent_attention(h, c, kr, W, p, mx, eps):
+def latent_attention(h, c, kr, W, p, mx, eps, rnd=exact):
     """windowed softmax attention over per-head keys [W_uk c, k_rot] and values W_uv c, gated and projected"""
     T, H, D, V = len(h), mx["heads"], mx["dim"], mx["vdim"]
-    qn, qr = latent_queries(h, W, p, mx, eps)
-    kn = (c @ W[p + "uk"].T).reshape(T, H, D)
-    v = (c @ W[p + "uv"].T).reshape(T, H, V)
+    qn, qr = latent_queries(h, W, p, mx, eps, rnd)
+    kn = rnd(c @ W[p + "uk"].T).reshape(T, H, D)
+    v = rnd(c @ W[p + "uv"].T).reshape(T, H, V)
     seen = window_mask(T, mx["mask"]["size"])
     o = np.empty((T, H, V))
     for j in range(H):
         s = (qn[:, j] @ kn[:, j].T + qr[:, j] @ kr.T) * mx["scale"]
-        o[:, j] = softmax_rows(s, seen) @ v[:, j]
+        o[:, j] = rnd(rnd(softmax_rows(s, seen)) @ v[:, j])
     gate = sigmoid(h @ W[p + "g"].T)
-    return (o.reshape(T, H * V) * gate) @ W[p + "o"].T
+    return rnd(o.reshape(T, H * V) * gate) @ W[p + "o"].T
 
 
-def dense_ff(h, W, p):
-    return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+def dense_ff(h, W, p, rnd=exact):
+    return rnd(silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
-def forward(cfg, W, tokens, layers_out=None):
+def forward(cfg, W, tokens, layers_out=None, rnd=exact):
     """logits [T, vocab] of every position of one sequence; layers_out receives x after each layer"""
     eps = cfg["norm"]["eps"]
     x = W["embed"][np.asarray(tokens)].astype(np.float64)
@@ -88,11 +96,12 @@ def forward(cfg, W, tokens, layers_out=None):
     for i, L in enumerate(cfg["layers"]):
         p, mx = "l%d." % i, L["mixer"]
         src = mx.get("kv_from")
-        held[i] = latent_kv(x, W, p + "mix.", mx, eps) if src is None else held[src]
-        y = latent_attention(x, held[i][0], held[i][1], W, p + "mix.", mx, eps)
+        h = rnd(x)
+        held[i] = latent_kv(h, W, p + "mix.", mx, eps, rnd) if src is None else held[src]
+        y = latent_attention(h, held[i][0], held[i][1], W, p + "mix.", mx, eps, rnd)
         x = x + rms_norm(y, W[p + "norm1"], eps)
         if L.get("mlp") is not None:
-            x = x + rms_norm(dense_ff(x, W, p + "mlp."), W[p + "norm2"], eps)
+            x = x + rms_norm(dense_ff(rnd(x), W, p + "mlp.", rnd), W[p + "norm2"], eps)
         if layers_out is not None:
             layers_out.append(x.copy())
-    return rms_norm(x, W["final.norm"], eps) @ W["embed"].T
+    return rnd(rms_norm(x, W["final.norm"], eps)) @ W["embed"].T

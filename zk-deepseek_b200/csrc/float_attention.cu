@@ -218,59 +218,61 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
             const int j0 = kt.lo + j * kTile;
             const int c_hi = pos - j0, c_lo = p.window > 0 ? c_hi - p.window + 1 : -1;
             const bool masked = __any_sync(0xffffffffu, c_hi < kTile - 1 || c_lo > 0);
-            float mx = -INFINITY;
+            float v[4][32];
 #pragma unroll
-            for (int c = 0; c < kTile; c += 32) {
-                float v[32];
-                tmem_ld32(tS + (uint32_t)c, v);
-                tmem_ld_wait();
-                if (masked) {
+            for (int q = 0; q < 4; ++q) tmem_ld32(tS + (uint32_t)(q * 32), v[q]);
+            tmem_ld_wait();
+            if (masked) {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i)
-                        if (c + i >= c_lo && c + i <= c_hi) mx = fmaxf(mx, v[i]);
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, v[i]);
-                }
+                for (int c = 0; c < kTile; ++c)
+                    if (c < c_lo || c > c_hi) v[c >> 5][c & 31] = -INFINITY;
             }
+            float mp[8];                              // independent chains: the warp has little else to issue
+#pragma unroll
+            for (int i = 0; i < 8; ++i) mp[i] = v[0][i];
+#pragma unroll
+            for (int c = 8; c < kTile; ++c) mp[c & 7] = fmaxf(mp[c & 7], v[c >> 5][c & 31]);
+            const float mx = fmaxf(fmaxf(fmaxf(mp[0], mp[1]), fmaxf(mp[2], mp[3])),
+                                   fmaxf(fmaxf(mp[4], mp[5]), fmaxf(mp[6], mp[7])));
             const float m_new = fmaxf(m_used, mx * p.scale_log2);
             if (j == kt.first[g]) {
                 m_used = m_new;
             } else if (__any_sync(0xffffffffu, m_new > m_used + 8.0f)) {
                 const float f = m_used == -INFINITY ? 0.f : exp2_approx(m_used - m_new);
                 for (int c = 0; c < p.dv; c += 32) {
-                    float v[32];
-                    tmem_ld32(tO + (uint32_t)c, v);
+                    float o[32];
+                    tmem_ld32(tO + (uint32_t)c, o);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] *= f;
-                    tmem_st32(tO + (uint32_t)c, v);
+                    for (int i = 0; i < 32; ++i) o[i] *= f;
+                    tmem_st32(tO + (uint32_t)c, o);
                 }
                 l *= f;
                 m_used = m_new;
             }
             const float m_sub = m_used == -INFINITY ? 0.f : m_used;
+            float lp[4] = {};
 #pragma unroll
-            for (int c = 0; c < kTile; c += 32) {
-                float v[32];
-                tmem_ld32(tS + (uint32_t)c, v);
-                tmem_ld_wait();
+            for (int q = 0; q < 4; ++q) {
                 uint32_t w[16];
+                if (q == 3) {                         // read again rather than held: registers
+                    tmem_ld32(tS + 96u, v[3]);
+                    tmem_ld_wait();
+                    if (masked) {
 #pragma unroll
-                for (int i = 0; i < 32; ++i) v[i] = exp2_approx(fmaf(v[i], p.scale_log2, -m_sub));
-                if (masked) {
-#pragma unroll
-                    for (int i = 0; i < 32; ++i)
-                        if (c + i < c_lo || c + i > c_hi) v[i] = 0.f;
+                        for (int i = 0; i < 32; ++i)
+                            if (96 + i < c_lo || 96 + i > c_hi) v[3][i] = -INFINITY;
+                    }
                 }
-                float part = 0.f;
 #pragma unroll
-                for (int i = 0; i < 32; ++i) part += v[i];
-                l += part;
+                for (int i = 0; i < 32; ++i) v[q][i] = exp2_approx(fmaf(v[q][i], p.scale_log2, -m_sub));
 #pragma unroll
-                for (int i = 0; i < 16; ++i) w[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
-                tmem_st16(tS + (uint32_t)(c / 2), w);
+                for (int i = 0; i < 32; ++i) lp[i & 3] += v[q][i];
+#pragma unroll
+                for (int i = 0; i < 16; ++i) w[i] = pack_bf16(v[q][2 * i], v[q][2 * i + 1]);
+                tmem_st16(tS + (uint32_t)(q * 16), w);
             }
+            l += (lp[0] + lp[1]) + (lp[2] + lp[3]);
             tmem_st_wait();
             tc_fence_before();
             __syncwarp();

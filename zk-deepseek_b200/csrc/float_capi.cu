@@ -55,16 +55,17 @@ int* fp_error_flag()
     return g_flag_dev[dev];
 }
 
-static constexpr long long kStreamRows = 16;     // up to here a linear layer streams its weights
+// up to here a linear layer streams its weights through the CUDA cores
+static constexpr long long kStreamRowsBf16 = 2, kStreamRowsF32 = 16;
 
 static bool linear_ok(const zkfp_linear_args* a)
 {
     if (!a || !a->A || !a->W || !a->out || a->M < 0 || a->N <= 0 || a->K <= 0) return false;
-    if ((a->N & 7) || (a->K & 7) || (a->lda & 7) || (a->ldw & 7) || (a->ldo & 3)) return false;
+    if ((a->N & 7) || (a->K & 7) || (a->lda & 7) || (a->ldw & 7) || (a->ldo & 7)) return false;
     if (a->lda < a->K || a->ldw < a->K || a->M > 0x7fffffffll || a->N > 0x7fffffffll || a->K > 0x7fffffffll) return false;
     if ((uintptr_t)a->A & 15 || (uintptr_t)a->W & 15 || (uintptr_t)a->out & 15) return false;
-    if (a->epilogue != ZKFP_EPI_GLU && ((a->ldo & 7) || a->ldo < a->N)) return false;
-    if (a->epilogue == ZKFP_EPI_GLU && a->ldo < a->N / 2) return false;
+    if (a->epilogue != ZKFP_EPI_GLU && a->ldo < a->N) return false;
+    if (a->epilogue == ZKFP_EPI_GLU && ((a->N & 15) || a->ldo < a->N / 2)) return false;
     if (a->epilogue == ZKFP_EPI_ROTATE &&
         (!a->table || !a->start || a->seq <= 0 || a->period <= 0 || (a->period & 1) || (a->offset & 1)))
         return false;
@@ -87,7 +88,7 @@ extern "C" {
 
 int zkfp_linear_path(const zkfp_linear_args* a)
 {
-    if (a->M <= kStreamRows) return 2;
+    if (a->M <= (a->dtype == ZKFP_BF16 ? kStreamRowsBf16 : kStreamRowsF32)) return 2;
     return a->dtype == ZKFP_BF16 ? 1 : 0;
 }
 
