@@ -3,9 +3,11 @@
 // attention_expanded_kernel (prefill): per-head keys [k1 | k2] and values.  A CTA owns one head and two tiles of 128
 // query tokens; keys come in tiles of 128.  Tensor memory holds both score tiles and both output tiles; the bfloat16
 // weights overwrite the scores they came from and feed the second product from tensor memory.  While one query tile is
-// in its softmax the tensor core works for the other.
+// in its softmax the tensor core works for the other.  Keys come through a ring of 64-column segments (16 KB), so that
+// the next tile starts to load as soon as the first segment of the current one has been used; values through whole
+// tiles, two where they fit.
 //   warp 0      TMA loads          warp 1      MMA issue
-//   warps 2-5   softmax, tile 0    warps 6-9   softmax, tile 1 (one query row per thread)
+//   warps 2-9   softmax, tile 0    warps 10-17 softmax, tile 1: two threads share a query row, half of the columns each
 // The running maximum only replaces the one in use when it has grown by more than 2^8; the output tile is then
 // rescaled in place.  A commit covers every MMA issued before it, so "scores ready" also says that the output tile is
 // free to be rescaled.
@@ -23,8 +25,10 @@ namespace {
 
 constexpr int kTile = 128;                     // query rows and keys per tile
 constexpr uint32_t kSeg = kTile * 128;         // bytes of 128 rows x 64 bfloat16
-constexpr int kThreadsAttn = 320;
-constexpr size_t kSmemMax = 226 * 1024;
+constexpr int kThreadsAttn = 576;
+constexpr int kMaxKeySlots = 8;
+constexpr int kHeadGroup = 32;
+constexpr size_t kSmemMax = 226 * 1024, kSmemAll = 227 * 1024;
 
 __device__ __forceinline__ float exp2_approx(float x)
 {
@@ -39,13 +43,15 @@ struct ExpandedParams {
     long long o_head;
     int seq, heads, base, window;
     int d1, d2, dv, seg1, seg2, segv;          // segments of 64 columns
-    int k_stages, v_stages;
+    int k_slots, v_stages;                     // ring of key segments, value tiles
     float scale_log2;                          // scale * log2(e)
+    uint32_t smem_bytes;
     int* error_flag;
 };
 
 struct ExpandedShared {
-    uint64_t q_full, k_full[4], k_empty[4], v_full[4], v_empty[4], s_full[2], p_full[2], o_full[2];
+    uint64_t q_full, k_full[kMaxKeySlots], k_empty[kMaxKeySlots], v_full[2], v_empty[2], s_full[2], p_full[2], o_full[2];
+    float row_max[2][2][kTile];            // [query tile][column half][row]; at the end the row sums
     uint32_t tmem;
     int abort;
 };
@@ -79,30 +85,41 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
                           const __grid_constant__ CUtensorMap tmK1, const __grid_constant__ CUtensorMap tmK2,
                           const __grid_constant__ CUtensorMap tmV, const ExpandedParams p)
 {
-    extern __shared__ uint8_t raw[];
+    // the tiles of the largest shapes leave less than a kilobyte, so the bookkeeping lies behind them in the same block
+    extern __shared__ __align__(1024) uint8_t raw[];
     uint8_t* base = (uint8_t*)(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
-    __shared__ ExpandedShared s;
+    const uint32_t tile_bytes = (uint32_t)(2 * (p.seg1 + p.seg2) + p.k_slots + p.v_stages * p.segv) * kSeg;
+    if (base + tile_bytes + sizeof(ExpandedShared) > raw + p.smem_bytes) {      // not the alignment the host counted on
+        if (threadIdx.x == 0) *(volatile int*)p.error_flag = 1;
+        return;
+    }
+    ExpandedShared& s = *reinterpret_cast<ExpandedShared*>(base + tile_bytes);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.y, t0 = (int)(gridDim.x - 1 - blockIdx.x) * 2 * kTile;    // longest blocks first
+    // the longest blocks of a group of heads first: short tails, keys and values of the group stay in L2
+    const int blocks = (p.seq + 2 * kTile - 1) / (2 * kTile), group0 = (int)blockIdx.x / (blocks * kHeadGroup) * kHeadGroup;
+    const int in_group = (int)blockIdx.x - group0 * blocks, width = min(kHeadGroup, p.heads - group0);
+    const int head = group0 + in_group % width, t0 = (blocks - 1 - in_group / width) * 2 * kTile;
     const int start = p.start[0];
     const KeyTiles kt = key_tiles(p, t0, start);
     const int segq = p.seg1 + p.seg2;
     const uint32_t sQ = smem_u32(base), bytesQ = (uint32_t)segq * kSeg;
-    const uint32_t sK = sQ + 2 * bytesQ, sV = sK + (uint32_t)p.k_stages * bytesQ, bytesV = (uint32_t)p.segv * kSeg;
+    const uint32_t sK = sQ + 2 * bytesQ, sV = sK + (uint32_t)p.k_slots * kSeg, bytesV = (uint32_t)p.segv * kSeg;
     volatile int* abort_flag = &s.abort;
 
     if (threadIdx.x == 0) {
         s.abort = 0;
         mbar_init(smem_u32(&s.q_full), 1);
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < kMaxKeySlots; ++i) {
             mbar_init(smem_u32(&s.k_full[i]), 1);
             mbar_init(smem_u32(&s.k_empty[i]), 1);
+        }
+        for (int i = 0; i < 2; ++i) {
             mbar_init(smem_u32(&s.v_full[i]), 1);
             mbar_init(smem_u32(&s.v_empty[i]), 1);
         }
         for (int g = 0; g < 2; ++g) {
             mbar_init(smem_u32(&s.s_full[g]), 1);
-            mbar_init(smem_u32(&s.p_full[g]), 4);
+            mbar_init(smem_u32(&s.p_full[g]), 8);
             mbar_init(smem_u32(&s.o_full[g]), 1);
         }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -127,17 +144,19 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
             }
             int ks = 0, vs = 0;
             uint32_t kp = 0, vp = 0;
-            for (int j = 0; j < kt.n; ++j) {
+            bool ok = true;
+            for (int j = 0; j < kt.n && ok; ++j) {
                 const int y = kt.lo - p.base + j * kTile;
-                if (!mbar_wait(smem_u32(&s.k_empty[ks]), kp ^ 1u, abort_flag)) break;
-                uint32_t bar = smem_u32(&s.k_full[ks]), dst = sK + (uint32_t)ks * bytesQ;
-                mbar_expect_tx(bar, bytesQ);
-                for (int c = 0; c < p.seg1; ++c) tma_load_3d(dst + c * kSeg, &tmK1, c * 64, head, y, bar);
-                for (int c = 0; c < p.seg2; ++c) tma_load_2d(dst + (p.seg1 + c) * kSeg, &tmK2, c * 64, y, bar);
-                if (++ks == p.k_stages) { ks = 0; kp ^= 1u; }
-                if (!mbar_wait(smem_u32(&s.v_empty[vs]), vp ^ 1u, abort_flag)) break;
-                bar = smem_u32(&s.v_full[vs]);
-                dst = sV + (uint32_t)vs * bytesV;
+                for (int c = 0; c < segq; ++c) {
+                    if (!(ok = mbar_wait(smem_u32(&s.k_empty[ks]), kp ^ 1u, abort_flag))) break;
+                    const uint32_t bar = smem_u32(&s.k_full[ks]), dst = sK + (uint32_t)ks * kSeg;
+                    mbar_expect_tx(bar, kSeg);
+                    if (c < p.seg1) tma_load_3d(dst, &tmK1, c * 64, head, y, bar);
+                    else tma_load_2d(dst, &tmK2, (c - p.seg1) * 64, y, bar);
+                    if (++ks == p.k_slots) { ks = 0; kp ^= 1u; }
+                }
+                if (!ok || !mbar_wait(smem_u32(&s.v_empty[vs]), vp ^ 1u, abort_flag)) break;
+                const uint32_t bar = smem_u32(&s.v_full[vs]), dst = sV + (uint32_t)vs * bytesV;
                 mbar_expect_tx(bar, bytesV);
                 for (int c = 0; c < p.segv; ++c) tma_load_3d(dst + c * kSeg, &tmV, c * 64, head, y, bar);
                 if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }
@@ -146,106 +165,110 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t idesc_s = idesc_bf16(kTile, kTile), idesc_o = idesc_bf16(kTile, (p.dv + 15) & ~15, true);
-            const int steps1 = (p.d1 + 15) / 16, steps2 = (p.d2 + 15) / 16;
             uint32_t pp[2] = {0, 0};
-            int ks = 0, vs = 0;
+            int ks = 0, vs = 0;                           // ring slot of the key tile's first segment, value stage
             uint32_t kp = 0, vp = 0;
-            auto scores = [&](int g) {
-                const uint32_t a = sQ + (uint32_t)g * bytesQ, b = sK + (uint32_t)ks * bytesQ, d = tmem + (uint32_t)g * kTile;
-                uint32_t acc = 0;
-                for (int k = 0; k < steps1 + steps2; ++k) {
-                    const int kk = k < steps1 ? k : p.seg1 * 4 + (k - steps1);       // 16-column step inside the tile
-                    const uint32_t off = (uint32_t)(kk >> 2) * kSeg + (uint32_t)(kk & 3) * 32u;
-                    umma_bf16(d, smem_desc_sw128(a + off), smem_desc_sw128(b + off), idesc_s, acc);
-                    acc = 1;
+            // the score product of query tile g with the key tile at (ks, kp); `load` waits for its segments,
+            // `release` hands each back after use
+            auto scores = [&](int g, bool use, bool load, bool release) {
+                const uint32_t a = sQ + (uint32_t)g * bytesQ, d = tmem + (uint32_t)g * kTile;
+                int slot = ks;
+                uint32_t phase = kp;
+                for (int c = 0; c < segq; ++c) {
+                    if (load) {
+                        if (!mbar_wait(smem_u32(&s.k_full[slot]), phase, abort_flag)) return false;
+                        tc_fence_after();
+                    }
+                    if (use) {
+                        const int cols = c < p.seg1 ? p.d1 - c * 64 : p.d2 - (c - p.seg1) * 64;
+                        const uint64_t ad = smem_desc_sw128(a + (uint32_t)c * kSeg), bd = smem_desc_sw128(sK + (uint32_t)slot * kSeg);
+#pragma unroll
+                        for (int k = 0; k < 4; ++k)
+                            if (k * 16 < cols) umma_bf16(d, ad + (uint64_t)(k * 2), bd + (uint64_t)(k * 2), idesc_s, (c | k) ? 1u : 0u);
+                    }
+                    if (release) umma_commit(smem_u32(&s.k_empty[slot]));
+                    if (++slot == p.k_slots) { slot = 0; phase ^= 1u; }
                 }
-                umma_commit(smem_u32(&s.s_full[g]));
+                if (use) umma_commit(smem_u32(&s.s_full[g]));
+                if (release) { ks = slot; kp = phase; }
+                return true;
             };
-            auto active = [&](int g, int j) { return j >= kt.first[g] && j <= kt.last[g]; };
+            auto active = [&](int g, int j) {
+                return g ? j >= kt.first[1] && j <= kt.last[1] : j >= kt.first[0] && j <= kt.last[0];
+            };
             bool ok = mbar_wait(smem_u32(&s.q_full), 0, abort_flag);
             for (int j = -1; j < kt.n && ok; ++j) {
                 if (j >= 0 && !(ok = mbar_wait(smem_u32(&s.v_full[vs]), vp, abort_flag))) break;
-                const bool next = j + 1 < kt.n;
-                bool k_ready = false;
                 for (int g = 0; g < 2 && ok; ++g) {
                     if (j >= 0 && active(g, j)) {
                         if (!(ok = mbar_wait(smem_u32(&s.p_full[g]), pp[g], abort_flag))) break;
                         pp[g] ^= 1u;
                         tc_fence_after();
                         const uint32_t a = tmem + (uint32_t)g * kTile, d = tmem + 256u + (uint32_t)g * kTile;
+                        const uint64_t vd = smem_desc_mn_sw128(sV + (uint32_t)vs * bytesV, kSeg);
+                        const bool opens = j == (g ? kt.first[1] : kt.first[0]);
 #pragma unroll
                         for (int k = 0; k < kTile / 16; ++k)
-                            umma_bf16_ts(d, a + (uint32_t)k * 8u,
-                                         smem_desc_mn_sw128(sV + (uint32_t)vs * bytesV + (uint32_t)k * 2048u, kSeg), idesc_o,
-                                         (j > kt.first[g] || k) ? 1u : 0u);
-                        if (j == kt.last[g]) umma_commit(smem_u32(&s.o_full[g]));
+                            umma_bf16_ts(d, a + (uint32_t)k * 8u, vd + (uint64_t)(k * 128), idesc_o, (!opens || k) ? 1u : 0u);
+                        if (j == (g ? kt.last[1] : kt.last[0])) umma_commit(smem_u32(&s.o_full[g]));
                     }
-                    if (next && active(g, j + 1)) {
-                        if (!k_ready) {
-                            if (!(ok = mbar_wait(smem_u32(&s.k_full[ks]), kp, abort_flag))) break;
-                            tc_fence_after();
-                            k_ready = true;
-                        }
-                        scores(g);
-                    }
+                    if (j >= 0 && g == 1) umma_commit(smem_u32(&s.v_empty[vs]));
+                    // every segment is waited for once and handed back once, also when no query tile uses it
+                    if (j + 1 < kt.n) ok = scores(g, active(g, j + 1), g == 0, g == 1);
                 }
-                // a stage is handed back only after its load has landed, also when no query tile used it
-                if (ok && next && !k_ready) ok = mbar_wait(smem_u32(&s.k_full[ks]), kp, abort_flag);
                 if (!ok) break;
-                if (j >= 0) {
-                    umma_commit(smem_u32(&s.v_empty[vs]));
-                    if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }
-                }
-                if (next) {
-                    umma_commit(smem_u32(&s.k_empty[ks]));
-                    if (++ks == p.k_stages) { ks = 0; kp ^= 1u; }
-                }
+                if (j >= 0 && ++vs == p.v_stages) { vs = 0; vp ^= 1u; }
             }
         }
     } else {
-        const int g = (warp - 2) >> 2, quarter = warp & 3, row = quarter * 32 + lane;
-        const int t = t0 + g * kTile + row, pos = start + t;
+        const int g = (warp - 2) >> 3, half = ((warp - 2) >> 2) & 1, quarter = warp & 3, row = quarter * 32 + lane;
+        const int t = t0 + g * kTile + row, pos = start + t, c0 = half * 64;
         const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
         const uint32_t tS = tmem + (uint32_t)g * kTile + lanes, tO = tmem + 256u + (uint32_t)g * kTile + lanes;
+        const int o_begin = half * ((p.dv / 2 + 31) & ~31), o_end = half ? p.dv : min(p.dv, (p.dv / 2 + 31) & ~31);
+        const int first_tile = g ? kt.first[1] : kt.first[0], last_tile = g ? kt.last[1] : kt.last[0];
+        auto pair_sync = [&] { asm volatile("bar.sync %0, 64;" ::"r"(1 + g * 4 + quarter) : "memory"); };
         float m_used = -INFINITY, l = 0.f;
         uint32_t sp = 0;
         bool ok = true;
-        for (int j = kt.first[g]; j <= kt.last[g]; ++j) {
-            if (!(ok = mbar_wait(smem_u32(&s.s_full[g]), sp, abort_flag))) break;
+        for (int j = first_tile; j <= last_tile; ++j) {
+            ok = mbar_wait(smem_u32(&s.s_full[g]), sp, abort_flag);
             sp ^= 1u;
             tc_fence_after();
+            float v[2][32];
+            tmem_ld32(tS + (uint32_t)c0, v[0]);
+            tmem_ld32(tS + (uint32_t)c0 + 32u, v[1]);
             // visible columns of this row: c_lo .. c_hi
-            const int j0 = kt.lo + j * kTile;
-            const int c_hi = pos - j0, c_lo = p.window > 0 ? c_hi - p.window + 1 : -1;
+            const int c_hi = pos - (kt.lo + j * kTile), c_lo = p.window > 0 ? c_hi - p.window + 1 : -1;
             const bool masked = __any_sync(0xffffffffu, c_hi < kTile - 1 || c_lo > 0);
-            float v[4][32];
-#pragma unroll
-            for (int q = 0; q < 4; ++q) tmem_ld32(tS + (uint32_t)(q * 32), v[q]);
             tmem_ld_wait();
             if (masked) {
 #pragma unroll
-                for (int c = 0; c < kTile; ++c)
-                    if (c < c_lo || c > c_hi) v[c >> 5][c & 31] = -INFINITY;
+                for (int c = 0; c < 64; ++c)
+                    if (c0 + c < c_lo || c0 + c > c_hi) v[c >> 5][c & 31] = -INFINITY;
             }
-            float mp[8];                              // independent chains: the warp has little else to issue
+            float mp[8];                              // independent chains
 #pragma unroll
             for (int i = 0; i < 8; ++i) mp[i] = v[0][i];
 #pragma unroll
-            for (int c = 8; c < kTile; ++c) mp[c & 7] = fmaxf(mp[c & 7], v[c >> 5][c & 31]);
-            const float mx = fmaxf(fmaxf(fmaxf(mp[0], mp[1]), fmaxf(mp[2], mp[3])),
-                                   fmaxf(fmaxf(mp[4], mp[5]), fmaxf(mp[6], mp[7])));
-            const float m_new = fmaxf(m_used, mx * p.scale_log2);
-            if (j == kt.first[g]) {
+            for (int c = 8; c < 64; ++c) mp[c & 7] = fmaxf(mp[c & 7], v[c >> 5][c & 31]);
+            const float mine = fmaxf(fmaxf(fmaxf(mp[0], mp[1]), fmaxf(mp[2], mp[3])),
+                                     fmaxf(fmaxf(mp[4], mp[5]), fmaxf(mp[6], mp[7])));
+            s.row_max[g][half][row] = mine;
+            // also: both threads of every row have read their scores before either overwrites any of them
+            pair_sync();
+            const float m_new = fmaxf(m_used, fmaxf(mine, s.row_max[g][half ^ 1][row]) * p.scale_log2);
+            if (j == first_tile) {
                 m_used = m_new;
-            } else if (__any_sync(0xffffffffu, m_new > m_used + 8.0f)) {
+            } else if (__any_sync(0xffffffffu, m_new > m_used + 8.0f)) {     // the same rows, so the same decision in both warps
                 const float f = m_used == -INFINITY ? 0.f : exp2_approx(m_used - m_new);
-                for (int c = 0; c < p.dv; c += 32) {
-                    float o[32];
-                    tmem_ld32(tO + (uint32_t)c, o);
+                for (int c = o_begin; c < o_end; c += 8) {
+                    int32_t o[8];
+                    tmem_ld8(tO + (uint32_t)c, o);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) o[i] *= f;
-                    tmem_st32(tO + (uint32_t)c, o);
+                    for (int i = 0; i < 8; ++i) o[i] = __float_as_int(__int_as_float(o[i]) * f);
+                    tmem_st8(tO + (uint32_t)c, o);
                 }
                 l *= f;
                 m_used = m_new;
@@ -253,24 +276,15 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
             const float m_sub = m_used == -INFINITY ? 0.f : m_used;
             float lp[4] = {};
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
+            for (int q = 0; q < 2; ++q) {
                 uint32_t w[16];
-                if (q == 3) {                         // read again rather than held: registers
-                    tmem_ld32(tS + 96u, v[3]);
-                    tmem_ld_wait();
-                    if (masked) {
-#pragma unroll
-                        for (int i = 0; i < 32; ++i)
-                            if (96 + i < c_lo || 96 + i > c_hi) v[3][i] = -INFINITY;
-                    }
-                }
 #pragma unroll
                 for (int i = 0; i < 32; ++i) v[q][i] = exp2_approx(fmaf(v[q][i], p.scale_log2, -m_sub));
 #pragma unroll
                 for (int i = 0; i < 32; ++i) lp[i & 3] += v[q][i];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) w[i] = pack_bf16(v[q][2 * i], v[q][2 * i + 1]);
-                tmem_st16(tS + (uint32_t)(q * 16), w);
+                tmem_st16(tS + (uint32_t)(half * 32 + q * 16), w);
             }
             l += (lp[0] + lp[1]) + (lp[2] + lp[3]);
             tmem_st_wait();
@@ -278,24 +292,25 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
             __syncwarp();
             if (lane == 0) mbar_arrive(smem_u32(&s.p_full[g]));
         }
-        if (ok && kt.first[g] <= kt.last[g] && mbar_wait(smem_u32(&s.o_full[g]), 0, abort_flag)) {
+        if (first_tile <= last_tile) {
+            pair_sync();                              // the last maxima have been read
+            s.row_max[g][half][row] = l;
+            pair_sync();
+            l += s.row_max[g][half ^ 1][row];
+        }
+        if (ok && first_tile <= last_tile && mbar_wait(smem_u32(&s.o_full[g]), 0, abort_flag)) {
             tc_fence_after();
             const float r = 1.0f / l;
             bf16* o = p.out + ((long long)t * p.heads + head) * p.o_head;
-            for (int c = 0; c < p.dv; c += 32) {
-                float v[32];
-                tmem_ld32(tO + (uint32_t)c, v);
+            for (int c = o_begin; c < o_end; c += 8) {
+                int32_t x[8];
+                tmem_ld8(tO + (uint32_t)c, x);
                 tmem_ld_wait();
                 if (t < p.seq) {
+                    float w[8];
 #pragma unroll
-                    for (int i = 0; i < 32; i += 8) {
-                        if (c + i < p.dv) {
-                            float w[8];
-#pragma unroll
-                            for (int k = 0; k < 8; ++k) w[k] = v[i + k] * r;
-                            store8(o + c + i, w);
-                        }
-                    }
+                    for (int k = 0; k < 8; ++k) w[k] = __int_as_float(x[k]) * r;
+                    store8(o + c, w);
                 }
             }
         }
@@ -307,17 +322,16 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
     if (threadIdx.x == 0 && s.abort) *(volatile int*)p.error_flag = 1;
 }
 
-size_t expanded_smem(const zkfp_attention_args& a, int& ks, int& vs)
+size_t expanded_smem(const zkfp_attention_args& a, int& k_slots, int& v_stages)
 {
     const size_t segq = (size_t)(a.d1 + 63) / 64 + (a.d2 + 63) / 64, segv = (a.dv + 63) / 64;
-    ks = vs = 1;
-    auto bytes = [&] { return 1024 + kSeg * ((2 + ks) * segq + vs * segv); };
-    if (bytes() > kSmemMax) return 0;
-    ++ks;
-    if (bytes() > kSmemMax) { --ks; return bytes(); }
-    ++vs;
-    if (bytes() > kSmemMax) --vs;
-    return bytes();
+    const size_t fixed = sizeof(ExpandedShared) + 512, segs = (kSmemAll - fixed) / kSeg;
+    if (segq > (size_t)kMaxKeySlots || 3 * segq + segv > segs) return 0;
+    v_stages = 3 * segq + 2 * segv <= segs ? 2 : 1;
+    const size_t left = segs - 2 * segq - v_stages * segv;
+    k_slots = (int)(left < (size_t)kMaxKeySlots ? left : (size_t)kMaxKeySlots);
+    const size_t bytes = kSeg * (2 * segq + k_slots + v_stages * segv) + fixed;
+    return bytes + 1024 < kSmemAll ? bytes + 1024 : kSmemAll;
 }
 
 }  // namespace
@@ -341,7 +355,7 @@ int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st)
     p.scale_log2 = a.scale * 1.4426950408889634f;
     p.error_flag = fp_error_flag();
     if (!p.error_flag) return ZKDS_ERR_WORKSPACE;
-    const size_t smem = expanded_smem(a, p.k_stages, p.v_stages);
+    const size_t smem = expanded_smem(a, p.k_slots, p.v_stages);
     CUtensorMap q1, q2, k1, k2, v;
     const uint64_t H = (uint64_t)a.heads, S = (uint64_t)a.seq, N = (uint64_t)a.keys;
     const uint64_t qs[2] = {(uint64_t)a.q_head * 2, (uint64_t)a.q_head * 2 * H};
@@ -355,11 +369,13 @@ int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st)
         !fp_tensor_map(&k1, a.k1, 3, dk1, ks, b3) || !fp_tensor_map(&k2, a.k2, 2, dk2, k2s, b2) ||
         !fp_tensor_map(&v, a.v, 3, dv, vs, b3))
         return ZKDS_ERR_UNSUPPORTED;
-    ZKDS_CUDA(cudaFuncSetAttribute(attention_expanded_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
+    ZKDS_CUDA(cudaFuncSetAttribute(attention_expanded_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemAll));
     // more than half the shared memory: one CTA per SM, so the tensor-memory allocation never waits
     const size_t want = smem < 120 * 1024 ? 120 * 1024 : smem;
-    const dim3 grid((unsigned)((a.seq + 2 * kTile - 1) / (2 * kTile)), (unsigned)a.heads);
-    attention_expanded_kernel<<<grid, kThreadsAttn, want, st>>>(q1, q2, k1, k2, v, p);
+    p.smem_bytes = (uint32_t)want;
+    const long long ctas = (a.seq + 2 * kTile - 1) / (2 * kTile) * a.heads;
+    if (ctas > 0x7fffffffll) return ZKDS_ERR_UNSUPPORTED;
+    attention_expanded_kernel<<<(unsigned)ctas, kThreadsAttn, want, st>>>(q1, q2, k1, k2, v, p);
     return fp_launched();
 }
 

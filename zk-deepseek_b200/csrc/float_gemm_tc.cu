@@ -265,7 +265,19 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
                     for (int c = c_begin; c < c_end; c += 32) {
                         if (m0 >= p.M || n0 + c >= p.N) break;
                         float v[32] = {};
-                        for (int k = 0; k < p.ksplit; ++k) {
+                        int k = 0;
+                        for (; k + 4 <= p.ksplit; k += 4) {      // four shares in flight, added in order
+                            float a[4][32];
+#pragma unroll
+                            for (int q = 0; q < 4; ++q)
+#pragma unroll
+                                for (int i = 0; i < 32; ++i) a[q][i] = __ldcg(src + (k + q) * step + (long long)(c + i) * kTM);
+#pragma unroll
+                            for (int q = 0; q < 4; ++q)
+#pragma unroll
+                                for (int i = 0; i < 32; ++i) v[i] += a[q][i];
+                        }
+                        for (; k < p.ksplit; ++k) {
 #pragma unroll
                             for (int i = 0; i < 32; ++i) v[i] += __ldcg(src + k * step + (long long)(c + i) * kTM);
                         }
