@@ -1425,11 +1425,329 @@ class MlaSmallWorkload(MlaWorkload):
         return MlaWorkload.cpu_sample(orc, np, seconds, rank)
 
 
+# --------------------------------------------------------------------------------------------
+# floating-point decoder designs
+# --------------------------------------------------------------------------------------------
+
+class OpTimer:
+    """Device time per call of named functions, given as (module or class, names).  Every step is queued behind a sleeping kernel, so
+    the events around a call see its kernels back to back and no launch gap."""
+
+    def __init__(self, torch, *owners):
+        self.torch, self.calls = torch, []
+        self.saved = [(o, n, getattr(o, n)) for o, names in owners for n in names]
+
+    def __enter__(self):
+        for o, n, fn in self.saved:
+            setattr(o, n, self._wrap(n, fn))
+        return self
+
+    def __exit__(self, *exc):
+        for o, n, fn in self.saved:
+            setattr(o, n, fn)
+        return False
+
+    def _wrap(self, name, fn):
+        def call(*a, **kw):
+            e0, e1 = (self.torch.cuda.Event(enable_timing=True) for _ in range(2))
+            e0.record()
+            out = fn(*a, **kw)
+            e1.record()
+            self.calls.append((name, a, e0, e1))
+            return out
+        return call
+
+    def run(self, step, reps=3):
+        """[(name, args, median seconds)] in call order"""
+        runs = []
+        for _ in range(reps):
+            self.calls = []
+            self.torch.cuda._sleep(40_000_000)
+            step()
+            self.torch.cuda.synchronize()
+            runs.append([e0.elapsed_time(e1) * 1e-3 for _, _, e0, e1 in self.calls])
+        return [(n, a, statistics.median(r[i] for r in runs)) for i, (n, a, _, _) in enumerate(self.calls)]
+
+
+class FloatDesignWorkload:
+    """Munalorn, a decoder with windowed latent attention and norms on the sublayers' outputs, random bfloat16 weights
+    at the sizes of a real model's layers: prefill of one 4096-token prompt through two layers of the largest size
+    (the second reads the first one's latents) and the output projection of the last position.  The line also holds
+    `sizes`: prefill and one-token decode at three sizes beside the integer model's dense block of the same sizes,
+    with the roofline fraction of every kernel class."""
+    name = "munalorn_prefill_4096"
+    metric = "munalorn_prefill_tokens_per_s"
+    unit = "tokens/s"
+    scaling = "weak"
+    dtype = "bf16"
+    T, VOCAB = 4096, 32768
+    #        width heads q_rank kv_rank ff
+    SIZES = {"w7168_h128": (7168, 128, 1536, 512, 18432), "w4096_h32": (4096, 32, 1024, 512, 14336),
+             "w2048_h16": (2048, 16, 768, 512, 8192)}
+    DIM, ROT, VDIM = 128, 64, 128
+
+    def __init__(self, torch, k, dev, rank):
+        self.torch, self.ik, self.dev = torch, k, dev
+        _b = importlib.import_module(PKG + ".build")
+        _b.build(library=_b.FLOAT_LIBRARY)
+        self.fm = importlib.import_module(PKG + ".float_model")
+        self.fc = importlib.import_module(PKG + ".float_config")
+        self.fk = importlib.import_module(PKG + ".float_kernel")
+        self.size = "w7168_h128"
+        self.model = self.build(self.size, self.T)
+        g = torch.Generator().manual_seed(3)
+        self.tok_host = torch.randint(0, self.VOCAB, (1, self.T), generator=g).pin_memory()
+        self.toks = self.tok_host.to(dev)
+        self.logits_host = torch.empty((1, self.VOCAB)).pin_memory()
+        n0 = self.fk.launches()
+        self.step()
+        self.launches_per_step = int(self.fk.launches() - n0)
+
+    def build(self, size, window, layers=2):
+        torch, (w, H, q, c, ff) = self.torch, self.SIZES[size]
+        cfg = {"architecture": "Munalorn", "vocab": self.VOCAB, "width": w, "norm": {"eps": 1e-6}, "layers": []}
+        for i in range(layers):
+            mx = {"heads": H, "dim": self.DIM, "rot_dim": self.ROT, "vdim": self.VDIM, "q_rank": q, "kv_rank": c,
+                  "scale": (self.DIM + self.ROT) ** -0.5, "mask": {"size": window},
+                  "rot": {"base": 10000.0, "dims": self.ROT}}
+            if i % 2:
+                mx["kv_from"] = i - 1
+            cfg["layers"].append({"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": ff}})
+        args = self.fc.parse_config(cfg)
+        args.max_seq_len, args.max_batch_size = self.T + 64, 1
+        g = torch.Generator(device=self.dev).manual_seed(1)
+
+        def weights(name, shape):
+            t = torch.randn(shape, generator=g, device=self.dev, dtype=torch.bfloat16)
+            return t * 0.1 + 1 if "norm" in name else (t if name == "embed" else t * shape[1] ** -0.5)
+        return self.fm.FloatTransformer(args).load_weights(weights, torch.device(self.dev))
+
+    def config(self):
+        w, H, q, c, ff = self.SIZES[self.size]
+        return {"workload": self.name, "model": "Munalorn (random weights)", "global_batch": 1, "seq_len": self.T,
+                "layers": 2, "width": w, "heads": H, "q_rank": q, "kv_rank": c, "ff": ff, "window": self.T,
+                "l2": "weights streamed per step (2.8 GB) far exceed L2"}
+
+    def prefill(self, model, toks, logits=True):
+        slots = model.begin_batch(1)
+        out = model.step(toks, 0, slots, want=None if logits else [])[0]
+        model.end_batch(slots)
+        return out
+
+    def step(self):
+        return self.prefill(self.model, self.toks)
+
+    def step_e2e(self):
+        self.logits_host.copy_(self.prefill(self.model, self.tok_host), non_blocking=True)
+        self.torch.cuda.current_stream().synchronize()
+
+    def e2e_bytes(self):
+        return self.tok_host.numel() * 8, self.logits_host.numel() * 4
+
+    def value(self, seconds_per_step, world):
+        return self.T * world / seconds_per_step
+
+    def check(self, orc):
+        """1 if a small prompt's logits are further from the float64 oracle than bfloat16 rounding explains"""
+        import numpy as np
+        from oracle import float_oracle as fo
+        torch = self.torch
+        mx = {"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 48, "q_rank": 56, "kv_rank": 72, "scale": 0.2,
+              "mask": {"size": 100}, "rot": {"base": 10000.0, "dims": 16}}
+        cfg = {"architecture": "Munalorn", "vocab": 256, "width": 160, "norm": {"eps": 1e-6},
+               "layers": [{"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": 200}}]}
+        args = self.fc.parse_config(cfg)
+        args.max_seq_len = 256
+        W, g = {}, torch.Generator().manual_seed(5)
+
+        def weights(name, shape):
+            t = torch.randn(shape, generator=g)
+            t = (t * 0.1 + 1 if "norm" in name else (t if name == "embed" else t * shape[1] ** -0.5)).to(torch.bfloat16)
+            W[name] = t.double().numpy()
+            return t
+        model = self.fm.FloatTransformer(args).load_weights(weights, torch.device(self.dev))
+        toks = torch.randint(0, 256, (1, 200), generator=g)
+        slots = model.begin_batch(1)
+        got = torch.cat([model.step(toks[:, :150], 0, slots, want=range(150))[0]] +
+                        [model.step(toks[:, p:p + 1], p, slots)[0] for p in range(150, 200)]).double().cpu().numpy()
+        want = fo.forward(cfg, W, toks[0].tolist())
+        self.fk.device_status(sync=True)
+        return int(np.sqrt(((got - want) ** 2).mean()) > 0.03 * want.std())
+
+    @staticmethod
+    def cpu_sample(orc, np, seconds, rank=0):
+        return None, None, 0
+
+    # ---- per-kernel fractions ----------------------------------------------------------------------------
+    OPS = ("linear", "attention", "perhead", "latent_post", "add_norm")
+
+    def float_classes(self, model, step, seq, start, peaks, decode):
+        """kernel class -> (seconds, fraction of its roofline) of one step"""
+        torch, out = self.torch, {}
+        graphs, self.fm.DECODE_GRAPHS = self.fm.DECODE_GRAPHS, False
+        try:
+            with OpTimer(torch, (self.fk, self.OPS)) as timer:
+                calls = timer.run(step)
+        finally:
+            self.fm.DECODE_GRAPHS = graphs
+        vis = self.visible(seq, start)
+        for name, a, sec in calls:
+            if name == "linear":
+                M, (N, Kd) = a[0].shape[0], a[1].shape
+                flops, nbytes = 2.0 * M * N * Kd, 2.0 * (N * Kd + M * (N + Kd))
+                if N == self.VOCAB:
+                    continue
+            elif name == "attention":
+                t = a[0]
+                flops = 2.0 * vis * t.heads * (t.d1 + t.d2 + t.dv)
+                nbytes = 2.0 * (start + seq) * (t.d1 + t.d2) * (1 if t.shared else t.heads) + \
+                    2.0 * seq * t.heads * (t.d1 + t.d2 + t.dv)
+            elif name == "perhead":
+                flops, nbytes = 2.0 * a[0].shape[0] * a[1].numel(), 2.0 * a[1].numel()
+            elif name == "add_norm":
+                flops, nbytes = 0.0, a[0].numel() * (4 + 4 + 4 + 2.0)
+            else:
+                flops, nbytes = 0.0, a[0].rows * (4.0 * a[0].ldy + 2 * (a[0].ldq + a[0].pitch))
+            o = out.setdefault(name, [0.0, 0.0])
+            o[0] += sec
+            o[1] += max(flops / (peaks["bf16_tflops"] * 1e12), nbytes / (peaks["hbm_gbs"] * 1e9))
+        return {n: {"us": round(s * 1e6, 1), "frac": round(r / s, 3)} for n, (s, r) in out.items()}
+
+    @staticmethod
+    def visible(seq, start):
+        return seq * start + seq * (seq + 1) / 2.0
+
+    def int_block(self, size):
+        """one dense block of the integer model at the same sizes (no window, no output gate)"""
+        torch, M = self.torch, importlib.import_module(PKG + ".model")
+        w, H, q, c, ff = self.SIZES[size]
+        a = M.ModelArgs(max_seq_len=self.T + 64, vocab_size=1024, dim=w, inter_dim=ff, n_layers=1, n_dense_layers=1,
+                        n_heads=H, q_lora_rank=q, kv_lora_rank=c, qk_nope_head_dim=self.DIM, qk_rope_head_dim=self.ROT,
+                        v_head_dim=self.VDIM)
+        M.world_size, M.rank, M.ACT_LIMBS = 1, 0, 3
+        g = torch.Generator(device=self.dev).manual_seed(7)
+        with torch.device(self.dev):
+            blk = M.Block(0, a)
+        for mod in blk.modules():
+            if isinstance(mod, M.RMSNorm_int):
+                mod.weight = (2**16 + _normal_i(torch, g, (mod.dim,), 2.0**8, self.dev, torch.int64)).to(torch.int32)
+            elif isinstance(mod, M.Linear_int):
+                mod.weight = _normal_i(torch, g, tuple(mod.weight.shape), 2.0**16 / math.sqrt(mod.weight.shape[1]), self.dev,
+                                       torch.int32)
+                mod.res_rescale = 16
+                if hasattr(mod, "scale"):
+                    mod.scale = torch.tensor(16, dtype=torch.int32, device=self.dev)
+        at = blk.attn
+        at.score_limbs, at.causal_skip = (3, 3), True
+        at.kv_cache[:, :self.T] = _normal_i(torch, g, (1, self.T, c), 2.0**16, self.dev, torch.int64)
+        at.pe_cache[:, :self.T] = _normal_i(torch, g, (1, self.T, self.ROT), 2.0**16, self.dev, torch.int64)
+        for n in ("softmax_init_q19", "silu_init_q23"):
+            getattr(self.ik, n)()
+        x = _normal_i(torch, g, (1, self.T, w), 2.0**16, self.dev, torch.int64)
+        freqs = M.precompute_freqs_cis(a).to(self.dev)
+        mask = torch.full((self.T, self.T), -(64 << 36), dtype=torch.int64, device=self.dev).triu_(1)
+        mask._zkds_causal = True
+        return (lambda: blk(x, 0, freqs[:self.T], mask)), (lambda: blk(x[:, :1], self.T, freqs[self.T:self.T + 1], None)), blk
+
+    INT_OPS = ("linear_prepared", "einsum_heads_prepared", "mla_scores_fused", "softmax_pv_fused", "glu_prepared",
+               "rms_norm_int64_device")
+
+    def int_classes(self, step, blk, seq, start, peaks):
+        """the same classes of the integer block, against its own arithmetic: int8 limb products at twice the
+        bfloat16 rate, bytes of the limb planes and of the int64 activations it moves"""
+        torch, K = self.torch, self.ik
+        with torch.inference_mode(), OpTimer(torch, (K, self.INT_OPS), (K.CachePlanes, ("scores", "softmax_pv"))) as timer:
+            calls = timer.run(step)
+        out, vis, at = {}, self.visible(seq, start), blk.attn
+        C, R, H = at.kv_lora_rank, at.qk_rope_head_dim, at.n_heads
+        for name, a, sec in calls:
+            if name in ("linear_prepared", "glu_prepared"):
+                pl = a[1] if name == "linear_prepared" else a[2]
+                M = seq
+                N, Kd = pl.N, pl.K
+                ops, nbytes = 2.0 * M * N * Kd * 3 * pl.limbs, float(pl.limbs) * N * Kd + 8.0 * M * (N + Kd)
+                cls = "linear"
+            elif name == "einsum_heads_prepared":
+                pl = a[1]
+                N, Kd = pl.N, pl.K
+                ops, nbytes = 2.0 * seq * H * N * Kd * 3 * pl.limbs, float(pl.limbs) * H * N * Kd
+                cls = "perhead"
+            elif name == "rms_norm_int64_device":
+                ops, nbytes, cls = 0.0, 16.0 * a[0].numel(), "norm"
+            else:
+                width = C + R if name in ("mla_scores_fused", "scores") else C
+                # every position's limb planes once (three limbs), beside the queries
+                ops, nbytes, cls = 2.0 * 9 * vis * H * width, 3.0 * (start + seq) * width + 8.0 * seq * H * width, "attention"
+            o = out.setdefault(cls, [0.0, 0.0])
+            o[0] += sec
+            o[1] += max(ops / (2 * peaks["bf16_tflops"] * 1e12), nbytes / (peaks["hbm_gbs"] * 1e9))
+        return {n: {"us": round(s * 1e6, 1), "frac": round(r / s, 3)} for n, (s, r) in out.items()}
+
+    def sizes(self, peaks):
+        torch, table = self.torch, {}
+        for size in self.SIZES:
+            model = self.model if size == self.size else self.build(size, self.T)
+            n = model.args.n_layers
+            row = {}
+            sec = _timed_steps(torch, _Step(lambda: self.prefill(model, self.toks, logits=False)), 10)
+            row["prefill_us_per_layer"] = round(sec / n * 1e6, 1)
+            row["prefill_kernels_of_%d_layers" % n] = self.float_classes(
+                model, lambda: self.prefill(model, self.toks, logits=False), self.T, 0, peaks, False)
+            slots = model.begin_batch(1)
+            model.step(self.toks, 0, slots, want=[])
+            one = self.toks[:, :1]
+
+            def decode():
+                model.step(one, self.T, slots)
+                model.cache.truncate(slots[0], self.T)
+            sec = _timed_steps(torch, _Step(decode), 30)
+            row["decode_us_per_step"] = round(sec * 1e6, 1)
+            row["decode_tokens_per_s"] = round(1 / sec, 1)
+            nbytes = 2.0 * sum(b.numel() for b in model.buffers() if b is not None and b.dtype == torch.bfloat16)
+            row["decode_frac_of_hbm"] = round(nbytes / (peaks["hbm_gbs"] * 1e9) / sec, 3)
+            row["decode_kernels_of_%d_layers" % n] = self.float_classes(model, decode, 1, self.T, peaks, True)
+            model.end_batch(slots)
+            if size == self.size:
+                self.model = None
+            del model
+            torch.cuda.empty_cache()
+            pre, dec, blk = self.int_block(size)
+            with torch.inference_mode():
+                sec = _timed_steps(torch, _Step(pre), 3)
+                row["integer_block_prefill_us_per_layer"] = round(sec * 1e6, 1)
+                row["integer_block_prefill_kernels"] = self.int_classes(pre, blk, self.T, 0, peaks)
+                sec = _timed_steps(torch, _Step(dec), 10)
+                row["integer_block_decode_us_per_layer"] = round(sec * 1e6, 1)
+                row["integer_block_decode_kernels"] = self.int_classes(dec, blk, 1, self.T, peaks)
+            del pre, dec, blk
+            torch.cuda.empty_cache()
+            table[size] = row
+        return {"sizes": table}
+
+    def roofline(self, peaks):
+        torch, fk = self.torch, self.fk
+        w, _, _, _, ff = self.SIZES[self.size]
+        W, A = self.model.layers[0].ff.w_gate_up, torch.randn(self.T, w, device=self.dev).to(torch.bfloat16)
+        out = torch.empty(self.T, ff, dtype=torch.bfloat16, device=self.dev)
+        sec = _timed_steps(torch, _Step(lambda: fk.linear(A, W, out, fk.GLU)), 10)
+        flops = 2.0 * self.T * w * 2 * ff
+        return {"bound": "tensor", "kernel": "linear_tc_kernel (gate | up with the GLU epilogue)",
+                "achieved": round(flops / sec / 1e12, 1), "peak": peaks["bf16_tflops"], "unit": "TFLOP/s",
+                "frac": round(flops / sec / 1e12 / peaks["bf16_tflops"], 4), "kernel_us": round(sec * 1e6, 1),
+                "traffic_note": "%d x %d x %d, source of the peak: %s" % (self.T, 2 * ff, w, peaks["source"])}
+
+
+class _Step:
+    def __init__(self, fn):
+        self.step = fn
+
+
 WORKLOADS = {"gemm": GemmWorkload, "gemm_prof": GemmProfWorkload, "gemm_cfg1": GemmSmallMWorkload,
              "gemm_wide": GemmWideRangeWorkload, "chain": ChainWorkload,
              "chain_prof": ChainProfWorkload, "mla": MlaWorkload, "mla_ref": MlaRefScaleWorkload,
              "mla_small": MlaSmallWorkload, "mla_causal": MlaCausalSkipWorkload, "moe": MoeWorkload,
-             "moe_small": MoeSmallWorkload, "decode": DecodeWorkload, "decode_sharded": DecodeShardedWorkload}
+             "moe_small": MoeSmallWorkload, "decode": DecodeWorkload, "decode_sharded": DecodeShardedWorkload,
+             "munalorn": FloatDesignWorkload}
 DEFAULT_WORKLOAD = "mla"
 
 
@@ -1616,7 +1934,8 @@ def main():
                          "CUDA time per operator and kernel to FILE (where a multi-rank step's time goes; the "
                          "timed numbers are taken before it)")
     ap.add_argument("--no-extras", action="store_true",
-                    help="default workload only: leave out the GEMM, small-M, reference-scale and reference-kernel parts")
+                    help="default workload: leave out the GEMM, small-M, reference-scale and reference-kernel parts; "
+                         "munalorn: leave out the table of sizes")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup
 
@@ -1733,6 +2052,8 @@ def main():
         wl.x_host = None
         extras = default_line_extras(torch, k, dev, rank, peaks, np, wl)
         extras["cpu_baseline_torch"] = torch_cpu_baseline(torch, np, 2.0)
+    if world == 1 and hasattr(wl, "sizes") and not args.no_extras:
+        extras = wl.sizes(peaks)
     if rank == 0:
         cpu_v, cpu_desc, _ = (wl.cpu_sample(orc, np, args.cpu_seconds)
                                 if world == 1 and args.cpu_seconds > 0 else (None, None, 0))
@@ -1740,7 +2061,7 @@ def main():
         line = {"metric": wl.metric, "value": round(wl.value(sec_per_step, world), 2), "unit": wl.unit,
                 "n_gpus": world, "steps": args.steps, "warmup": args.warmup,
                 "ms_per_step": round(sec_per_step * 1e3, 4), "higher_is_better": True,
-                "scaling": getattr(wl, "scaling", "weak"), "vs_baseline": None, "dtype": "int64",
+                "scaling": getattr(wl, "scaling", "weak"), "vs_baseline": None, "dtype": getattr(wl, "dtype", "int64"),
                 "data": "synthetic", "config": wl.config(),
                 "e2e": {"value": round(wl.value(e2e_sec, world), 2), "unit": wl.unit,
                         "h2d_bytes_per_step": h2d, "d2h_bytes_per_step": d2h,

@@ -147,7 +147,8 @@ def plain_attention(q, k, v, start, base, window, scale):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("S,start,H,D,R,V,window", [
     (17, 0, 2, 64, 32, 64, 90), (130, 0, 1, 64, 32, 64, 0), (300, 50, 3, 48, 16, 80, 130), (300, 0, 2, 64, 32, 64, 7),
-    (257, 90, 2, 40, 24, 56, 1), (513, 700, 1, 128, 64, 128, 257), (260, 5, 2, 128, 64, 120, 100000), (385, 128, 1, 16, 8, 16, 129)])
+    (257, 90, 2, 40, 24, 56, 1), (513, 700, 1, 128, 64, 128, 257), (260, 5, 2, 128, 64, 120, 100000), (385, 128, 1, 16, 8, 16, 129),
+    (150, 20, 2, 64, 32, 168, 77), (90, 0, 1, 456, 64, 64, 50)])
 def test_expanded_attention(K, dtype, S, start, H, D, R, V, window):
     dt = getattr(torch, dtype)
     base = max(0, start - window + 1) if window else 0
@@ -164,7 +165,8 @@ def test_expanded_attention(K, dtype, S, start, H, D, R, V, window):
                        k1_tok=kv.stride(0), k1_head=D, k2_tok=kr.stride(0), v_tok=kv.stride(0), v_head=V, base=base,
                        keys=keys, batch=1, seq=S, heads=H, d1=D, d2=R, dv=V, window=window, shared=0, dtype=K.code(dt),
                        scale=(D + R) ** -0.5, max_keys=keys)
-    assert K.attention_path(ctypes.byref(a)) == (1 if dtype == "bfloat16" else 0)
+    fits = V <= 128 and D <= 320                  # wider heads run on the CUDA cores
+    assert K.attention_path(ctypes.byref(a)) == (1 if dtype == "bfloat16" and fits else 0)
     K.attention(a)
     q64, kv64, kr64 = (t.double().cpu().numpy() for t in (q, kv, kr))
     k = np.concatenate([kv64[:, :H * D].reshape(keys, H, D), np.repeat(kr64[:, None, :R], H, 1)], 2)
@@ -178,7 +180,7 @@ def test_expanded_attention(K, dtype, S, start, H, D, R, V, window):
 @pytest.mark.parametrize("starts,S,H,C,R,window", [
     ([0], 1, 4, 64, 32, 90), ([255], 1, 4, 64, 32, 64), ([256], 1, 4, 64, 32, 65), ([100], 2, 5, 64, 32, 90),
     ([77], 16, 16, 64, 32, 40), ([5, 130], 3, 24, 128, 64, 64), ([1000], 1, 128, 512, 64, 513), ([700], 5, 48, 512, 64, 0),
-    ([0, 63, 64], 1, 5, 72, 40, 65), ([300], 1, 8, 24, 8, 1)])
+    ([0, 63, 64], 1, 5, 72, 40, 65), ([300], 1, 8, 24, 8, 1), ([130], 2, 3, 520, 64, 100)])
 def test_latent_attention(K, dtype, starts, S, H, C, R, window):
     dt, B, P, cap = getattr(torch, dtype), len(starts), C + R, max(starts) + S + 9
     cache, q = rnd((B + 2, cap, P), dtype), rnd((B * S, H, P), dtype, 1)
@@ -195,7 +197,7 @@ def test_latent_attention(K, dtype, starts, S, H, C, R, window):
                        q_head=P, o_head=C, k1_tok=P, k2_tok=P, v_tok=P, slot_stride=cache.stride(0), keys=cap, batch=B, seq=S,
                        heads=H, d1=C, d2=R, dv=C, window=window, shared=1, dtype=K.code(dt), scale=P ** -0.5,
                        max_keys=min(max(starts) + S, window + S - 1) if window else max(starts) + S)
-    assert K.attention_path(ctypes.byref(a)) == (1 if dtype == "bfloat16" else 0)
+    assert K.attention_path(ctypes.byref(a)) == (1 if dtype == "bfloat16" and C <= 512 else 0)
     n = K.attention_scratch(a)
     scratch = torch.full((max(n, 1),), float("nan"), device="cuda")      # nothing may be read before it is written
     a.scratch = scratch.data_ptr()

@@ -566,6 +566,20 @@ def test_resident_checkpoint_loader(M, kmod, dev, tmp_path):
     want = G.generate(model, prompts, 3, eos_id=-5, temperature=0.0)
     got = G.generate(loaded, prompts, 3, eos_id=-5, temperature=0.0)
     assert got == want
+    # the same directory through the registry, and its steps through the trace replayer
+    import dataclasses
+    import json
+    pkg = M.__name__.rsplit(".", 1)[0]
+    registry, trace = (importlib.import_module(pkg + "." + n) for n in ("registry", "trace"))
+    with open(os.path.join(ck, "config.json"), "w") as f:
+        json.dump(dataclasses.asdict(a), f)
+    reg = registry.load(ck, max_seq_len=a.max_seq_len)
+    assert isinstance(reg, M.Transformer) and G.generate(reg, prompts, 3, eos_id=-5, temperature=0.0) == want
+    rp = trace.Replayer(reg)
+    logits = rp.entry("a", prompts[0], [1, 3])
+    assert logits.shape == (2, a.vocab_size) and int(logits[1].argmax()) == want[0][0]
+    assert int(rp.entry("a", [want[0][0]], [0])[0].argmax()) == want[0][1]
+    rp.end("a")
     kmod.device_status()
 
 

@@ -555,13 +555,13 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid_c
     if (threadIdx.x == 0 && s.abort) *(volatile int*)p.error_flag = 1;
 }
 
-// merges the chunks of 32 rows x 32 latent columns.  grid (c / 32, row tiles * 4, batch)
+// merges the chunks of 32 rows x 8 latent columns: the warps share the chunks.  grid (c / 8, row tiles * 4, batch)
 __global__ void __launch_bounds__(256)
 latent_combine_kernel(const LatentParams p, bf16* __restrict__ out, long long o_head)
 {
-    __shared__ float tile[32][33];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.z;
-    const int rt = blockIdx.y >> 2, row = (blockIdx.y & 3) * 32 + lane, row0 = rt * kTile, c0 = blockIdx.x * 32;
+    __shared__ float red[8][9][32];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.z, c0 = blockIdx.x * 8;
+    const int rt = blockIdx.y >> 2, row = (blockIdx.y & 3) * 32 + lane, row0 = rt * kTile;
     if (row0 + (int)(blockIdx.y & 3) * 32 >= p.rows) return;
     int first, n;
     chunk_range(p.start[b], row0, p.rows, p.heads, p.window, first, n);
@@ -570,29 +570,38 @@ latent_combine_kernel(const LatentParams p, bf16* __restrict__ out, long long o_
     const bool row_ok = row0 + row < p.rows;
     float m = -INFINITY;
     if (row_ok)
-#pragma unroll 8
-        for (int i = 0; i < n; ++i) m = fmaxf(m, ml[(long long)i * 256]);
-    float acc[4] = {}, l = 0.f;
-    const int c = c0 + warp * 4;
-    if (row_ok && c < p.c) {
-        const float* src = p.part + (t0 * p.c + c) * 128 + row;
 #pragma unroll 4
-        for (int i = 0; i < n; ++i) {
+        for (int i = warp; i < n; i += 8) m = fmaxf(m, ml[(long long)i * 256]);
+    red[warp][0][lane] = m;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 8; ++k) m = fmaxf(m, red[k][0][lane]);
+    __syncthreads();
+    float acc[8] = {}, l = 0.f;
+    if (row_ok) {
+        const float* src = p.part + (t0 * p.c + c0) * 128 + row;
+#pragma unroll 4
+        for (int i = warp; i < n; i += 8) {
             const float w = exp2_approx(ml[(long long)i * 256] - m);
             l = fmaf(w, ml[(long long)i * 256 + 128], l);
 #pragma unroll
-            for (int k = 0; k < 4; ++k) acc[k] = fmaf(w, src[((long long)i * p.c + k) * 128], acc[k]);
+            for (int k = 0; k < 8; ++k) acc[k] = fmaf(w, src[((long long)i * p.c + k) * 128], acc[k]);
         }
     }
-    const float r = 1.0f / l;
 #pragma unroll
-    for (int k = 0; k < 4; ++k) tile[warp * 4 + k][lane] = acc[k] * r;
+    for (int k = 0; k < 8; ++k) red[warp][k][lane] = acc[k];
+    red[warp][8][lane] = l;
     __syncthreads();
-    for (int i = warp; i < 32; i += 8) {
-        const int rr = row0 + (int)(blockIdx.y & 3) * 32 + i;
-        if (rr < p.rows && c0 + lane < p.c)
-            out[((long long)b * p.rows + rr) * o_head + c0 + lane] = __float2bfloat16_rn(tile[lane][i]);
+    // thread (row, column): eight threads write the 16 bytes of a row
+    const int rr = threadIdx.x >> 3, k = threadIdx.x & 7;
+    float v = 0.f, sum = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+        v += red[w][k][rr];
+        sum += red[w][8][rr];
     }
+    const int r = row0 + (int)(blockIdx.y & 3) * 32 + rr;
+    if (r < p.rows) out[((long long)b * p.rows + r) * o_head + c0 + k] = __float2bfloat16_rn(v / sum);
 }
 
 int latent_chunks(const zkfp_attention_args& a) { return (a.max_keys + kChunk - 1) / kChunk + 1; }
@@ -649,7 +658,7 @@ int launch_attention_decode_tc(const zkfp_attention_args& a, cudaStream_t st)
                                                                                                              k2, p);
     int rc = fp_launched();
     if (rc != ZKDS_OK) return rc;
-    latent_combine_kernel<<<dim3((unsigned)((p.c + 31) / 32), (unsigned)p.row_tiles * 4, (unsigned)a.batch), 256, 0, st>>>(
+    latent_combine_kernel<<<dim3((unsigned)(p.c / 8), (unsigned)p.row_tiles * 4, (unsigned)a.batch), 256, 0, st>>>(
         p, (bf16*)a.out, a.o_head);
     return fp_launched();
 }

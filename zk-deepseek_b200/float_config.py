@@ -90,7 +90,11 @@ def _latent_attention(i, mx, shapes, layers):
         if not 0 <= kv_from < i or layers[kv_from].mixer.kv_from is not None:
             raise ConfigError("layer %d reads the latents of layer %d, which has none of its own" % (i, kv_from))
     H = int(mx["heads"])
-    rot = mx.get("rot") or {}
+    rot = mx.get("rot")
+    if rot is None and kv_from is not None:
+        rot = {"base": layers[kv_from].mixer.rot.base, "dims": layers[kv_from].mixer.rot.dims}
+    if not rot:
+        raise ConfigError("layer %d has no rotation" % i)
     rot_dim = int(mx["rot_dim"]) if mx.get("rot_dim") is not None else int(rot["dims"])
     rotary = Rotary(float(rot["base"]), int(rot.get("dims", rot_dim)))
     if rotary.dims != rot_dim or rot_dim % 2:

@@ -992,8 +992,12 @@ class Transformer(nn.Module):
         return self.layers[layer_id](h, start_pos, freqs_cis, mask)
 
     @torch.inference_mode()
-    def finish_inference(self, h):
-        h = self.norm(h)[0][:, -1].contiguous()          # last position of every sequence: [B, dim]
+    def finish_inference(self, h, want=None):
+        h = self.norm(h)[0]
+        if want is None:
+            h = h[:, -1].contiguous()                    # last position of every sequence: [B, dim]
+        else:
+            h = h.reshape(-1, h.shape[-1])[list(want)].contiguous()
         logits = self.head(h[None, :])      # [1, B, vocab] (B = 1 in the reference)
         if world_size > 1:
             logits = _all_gather_last(logits)
@@ -1014,7 +1018,7 @@ class Transformer(nn.Module):
     def end_batch(self, batch):
         pass
 
-    def _forward_step(self, toks, prev_pos, layer_probe):
+    def _forward_step(self, toks, prev_pos, layer_probe, want=None):
         """one pass over all layers; finish_inference raises ZkdsError if a kernel flagged its operands"""
         h, start_pos, seqlen = self.prep_inference(toks, prev_pos)
         layer_tokens = []
@@ -1023,18 +1027,19 @@ class Transformer(nn.Module):
             if layer_probe:
                 probe = self.head(self.norm(h)[0][:, -1].contiguous()[None, :])
                 layer_tokens.append(probe.argmax(dim=-1).view(-1).tolist())
-        return self.finish_inference(h), layer_tokens
+        return self.finish_inference(h, want), layer_tokens
 
     @torch.inference_mode()
-    def step(self, toks, prev_pos, batch=None, layer_probe=False):
-        """(logits of the last position, info): runs toks [B, S] of sequences that stand at prev_pos, writes the
-        step's tokens.bin under `snark`"""
+    def step(self, toks, prev_pos, batch=None, want=None, layer_probe=False):
+        """(logits, info): runs toks [B, S] of sequences that stand at prev_pos, writes the step's tokens.bin under
+        `snark`.  want: rows b * S + s whose logits are returned, None the last of every sequence"""
+        toks = toks.to(self.device)
         if snark:
             os.makedirs(f"{zkDataDir}/pos_{prev_pos}", exist_ok=True)
             saveTensor(f"{zkDataDir}/pos_{prev_pos}/tokens.bin", toks[0].cpu())
         info = {}
         try:
-            logits, layer_tokens = self._forward_step(toks, prev_pos, layer_probe)
+            logits, layer_tokens = self._forward_step(toks, prev_pos, layer_probe, want)
         except K.ZkdsError as err:
             if err.status != K.ERR_RANGE:
                 raise
@@ -1042,7 +1047,7 @@ class Transformer(nn.Module):
             # numbers are wrong.  The step only wrote cache rows it owns, so it is simply run again with every
             # limb count measured on the device.
             with measured_limbs(self):
-                logits, layer_tokens = self._forward_step(toks, prev_pos, layer_probe)
+                logits, layer_tokens = self._forward_step(toks, prev_pos, layer_probe, want)
             info["rerun_measured"] = True
         if layer_probe:
             info["layer_tokens"] = layer_tokens

@@ -9,6 +9,7 @@ import importlib
 import json
 import os
 import struct
+import sys
 
 try:
     from . import build as _build
@@ -90,9 +91,10 @@ def load_float_model(model_dir, dtype="bfloat16", device="cuda", max_seq_len=409
     _build.build(library=_build.FLOAT_LIBRARY)
     fm = _module("float_model")
     model = fm.FloatTransformer(args, getattr(torch, dtype) if isinstance(dtype, str) else dtype)
-    unknown = sorted(set(files.where) - set(model.tensor_names()))
-    if unknown:
-        raise ValueError("the checkpoint holds tensors the configuration has no place for: %s" % ", ".join(unknown[:5]))
+    unused = sorted(set(files.where) - set(model.tensor_names()))
+    if unused:
+        print("tensors the configuration has no place for: %s%s" % (", ".join(unused[:5]), " ..." if unused[5:] else ""),
+              file=sys.stderr)
     return model.load_weights(files, torch.device(device))
 
 

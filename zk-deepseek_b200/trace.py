@@ -35,7 +35,7 @@ class Replayer:
         toks = torch.tensor([tokens], dtype=torch.int64)
         logits, _ = self.model.step(toks, req[1], req[0], want=want)
         req[1] += len(tokens)
-        return logits.float().cpu()
+        return logits.reshape(-1, logits.shape[-1]).float().cpu()
 
     def end(self, rid):
         slots, _ = self.open.pop(rid)
