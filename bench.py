@@ -1584,12 +1584,8 @@ class FloatDesignWorkload:
     def float_classes(self, model, step, seq, start, peaks, decode):
         """kernel class -> (seconds, fraction of its roofline) of one step"""
         torch, out = self.torch, {}
-        graphs, self.fm.DECODE_GRAPHS = self.fm.DECODE_GRAPHS, False
-        try:
-            with OpTimer(torch, (self.fk, self.OPS)) as timer:
-                calls = timer.run(step)
-        finally:
-            self.fm.DECODE_GRAPHS = graphs
+        with OpTimer(torch, (self.fk, self.OPS)) as timer:
+            calls = timer.run(step)
         vis = self.visible(seq, start)
         for name, a, sec in calls:
             if name == "linear":

@@ -32,6 +32,7 @@ typedef struct {
     long long lda, ldw, ldo, ldaux;
     long long M, N, K;     /* N, K padded (GLU: N a multiple of 16) */
     long long seq;         /* rotate: rows per sequence */
+    long long positions;   /* rotate: rows of the table; a position outside them leaves its row unrotated */
     int dtype, out_dtype, epilogue;
     int pairs, period, offset;
 } zkfp_linear_args;

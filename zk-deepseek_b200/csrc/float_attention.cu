@@ -395,7 +395,7 @@ struct LatentParams {
     const int* slots;
     float* part;               // [batch][row tile][chunk][c][128]
     float* ml;                 // [batch][row tile][chunk][2][128]: maximum (log2 units), sum
-    int rows, heads, seq, window, c, r, segc, segr, chunks, row_tiles;
+    int rows, heads, seq, window, c, r, segc, segr, chunks, row_tiles, keys;
     float scale_log2;
     int* error_flag;
 };
@@ -426,6 +426,10 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid_c
     const int b = blockIdx.z, row0 = blockIdx.y * kTile, start = p.start[b];
     int first, n;
     chunk_range(start, row0, p.rows, p.heads, p.window, first, n);
+    if (start < 0 || start + p.seq > p.keys || n > p.chunks) {        // not a step of this cache
+        if (threadIdx.x == 0) *(volatile int*)p.error_flag = 1;
+        return;
+    }
     if ((int)blockIdx.x >= n) return;
     const int j0 = (first + (int)blockIdx.x) * kChunk;
     uint8_t* base = (uint8_t*)(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
@@ -565,6 +569,7 @@ latent_combine_kernel(const LatentParams p, bf16* __restrict__ out, long long o_
     if (row0 + (int)(blockIdx.y & 3) * 32 >= p.rows) return;
     int first, n;
     chunk_range(p.start[b], row0, p.rows, p.heads, p.window, first, n);
+    if (p.start[b] < 0 || p.start[b] + p.seq > p.keys || n > p.chunks) return;
     const long long t0 = ((long long)b * p.row_tiles + rt) * p.chunks;
     const float* ml = p.ml + t0 * 256 + row;
     const bool row_ok = row0 + row < p.rows;
@@ -635,6 +640,7 @@ int launch_attention_decode_tc(const zkfp_attention_args& a, cudaStream_t st)
     p.rows = (int)(a.seq * a.heads); p.heads = (int)a.heads; p.seq = (int)a.seq; p.window = a.window;
     p.c = a.d1; p.r = a.d2; p.segc = (a.d1 + 63) / 64; p.segr = (a.d2 + 63) / 64;
     p.chunks = latent_chunks(a);
+    p.keys = (int)a.keys;
     p.row_tiles = (p.rows + kTile - 1) / kTile;
     p.part = a.scratch;
     p.ml = a.scratch + (long long)a.batch * p.row_tiles * p.chunks * 128 * p.c;

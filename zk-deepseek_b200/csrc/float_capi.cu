@@ -67,7 +67,7 @@ static bool linear_ok(const zkfp_linear_args* a)
     if (a->epilogue != ZKFP_EPI_GLU && a->ldo < a->N) return false;
     if (a->epilogue == ZKFP_EPI_GLU && ((a->N & 15) || a->ldo < a->N / 2)) return false;
     if (a->epilogue == ZKFP_EPI_ROTATE &&
-        (!a->table || !a->start || a->seq <= 0 || a->period <= 0 || (a->period & 1) || (a->offset & 1)))
+        (!a->table || !a->start || a->seq <= 0 || a->positions <= 0 || a->positions > 0x7fffffffll || a->period <= 0 || (a->period & 1) || (a->offset & 1)))
         return false;
     if (a->epilogue == ZKFP_EPI_GATE && (!a->aux || (a->ldaux & 7) || ((uintptr_t)a->aux & 15))) return false;
     return a->epilogue >= 0 && a->epilogue <= ZKFP_EPI_GLU && (a->dtype | a->out_dtype) <= 1;
@@ -98,7 +98,7 @@ int zkfp_linear(const zkfp_linear_args* a, void* stream)
     if (a->M == 0) return ZKDS_OK;
     LinEpi e;
     e.out = a->out; e.aux = a->aux; e.table = (const float2*)a->table; e.start = a->start;
-    e.ldo = a->ldo; e.ldaux = a->ldaux; e.seq = a->seq > 0 ? a->seq : 1;
+    e.ldo = a->ldo; e.ldaux = a->ldaux; e.seq = a->seq > 0 ? a->seq : 1; e.positions = a->positions;
     e.kind = a->epilogue; e.out_bf16 = a->out_dtype; e.aux_bf16 = a->dtype;
     e.pairs = a->pairs; e.period = a->period > 0 ? a->period : 1; e.offset = a->offset;
     cudaStream_t st = (cudaStream_t)stream;

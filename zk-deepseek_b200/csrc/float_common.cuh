@@ -11,6 +11,8 @@ namespace zkds {
 
 using bf16 = __nv_bfloat16;
 
+constexpr int kSharedMax = 227 * 1024;  // dynamic shared memory a CTA may ask for
+
 int fp_sm_count();
 int fp_launched();                      // cudaGetLastError -> status, counts the launch
 int* fp_error_flag();                   // device view of the host-mapped word that bounded waits set
@@ -91,7 +93,7 @@ struct LinEpi {
     const void* aux;
     const float2* table;
     const int* start;
-    long long ldo, ldaux, seq;
+    long long ldo, ldaux, seq, positions;
     int kind, out_bf16, aux_bf16;
     int pairs, period, offset;
 };
@@ -111,7 +113,7 @@ __device__ __forceinline__ int epi_position(const LinEpi& e, long long m)
 __device__ __forceinline__ void rotate_pair(const LinEpi& e, int pos, int n, float& u, float& v)
 {
     const int w = n % e.period - e.offset;
-    if (w < 0 || (w >> 1) >= e.pairs) return;
+    if (w < 0 || (w >> 1) >= e.pairs || (unsigned)pos >= (unsigned)e.positions) return;
     const float2 cs = e.table[(long long)pos * e.pairs + (w >> 1)];
     const float a = u * cs.x - v * cs.y;
     v = v * cs.x + u * cs.y;

@@ -26,6 +26,7 @@ constexpr int kThreadsTc = 64 + 32 * kEpiWarps;
 constexpr int kMaxStages = 12;
 constexpr uint32_t kBytesA = kTM * kBK * 2;
 constexpr uint32_t kStageBlock = 32 * 32 * 4;      // staging per epilogue warp
+constexpr int kLinearSmemMax = 226 * 1024;         // leaves room for the static part
 
 struct TcParams {
     int M, N, NT, kblocks, stages;
@@ -336,7 +337,7 @@ bool fp_tensor_map(CUtensorMap* map, const void* base, int rank, const uint64_t*
 
 // partial sums and arrival counters of split launches: one block per device, allocated at first use (calls on
 // several streams of one device must not overlap, like every call that uses library-owned scratch)
-static bool split_workspace(int pairs, float** partial, unsigned** counter)
+static bool split_workspace(int pairs, float** partial, unsigned** counter, cudaStream_t st)
 {
     static struct { float* p; unsigned* c; } ws[64];
     int dev = 0;
@@ -345,7 +346,7 @@ static bool split_workspace(int pairs, float** partial, unsigned** counter)
         void *a = nullptr, *b = nullptr;
         const size_t bytes_c = (size_t)pairs * 2 * kEpiWarps * sizeof(unsigned);
         if (cudaMalloc(&a, (size_t)pairs * 2 * 256 * kTM * sizeof(float)) != cudaSuccess) return false;
-        if (cudaMalloc(&b, bytes_c) != cudaSuccess || cudaMemset(b, 0, bytes_c) != cudaSuccess) return false;
+        if (cudaMalloc(&b, bytes_c) != cudaSuccess || cudaMemsetAsync(b, 0, bytes_c, st) != cudaSuccess) return false;
         ws[dev].p = (float*)a;
         ws[dev].c = (unsigned*)b;
     }
@@ -389,7 +390,7 @@ int launch_linear_tc(const zkfp_linear_args& a, const LinEpi& e, cudaStream_t st
     p.kb_per_split = (p.kblocks + p.ksplit - 1) / p.ksplit;
     p.partial = nullptr;
     p.counter = nullptr;
-    if (p.ksplit > 1 && !split_workspace(pairs, &p.partial, &p.counter)) return ZKDS_ERR_WORKSPACE;
+    if (p.ksplit > 1 && !split_workspace(pairs, &p.partial, &p.counter, st)) return ZKDS_ERR_WORKSPACE;
     p.stages = (int)((192u * 1024u) / stage_bytes);
     if (p.stages > kMaxStages) p.stages = kMaxStages;
     CUtensorMap tmA, tmW;
@@ -398,7 +399,8 @@ int launch_linear_tc(const zkfp_linear_args& a, const LinEpi& e, cudaStream_t st
     const uint32_t ba[2] = {kBK, kTM}, bw[2] = {kBK, (uint32_t)p.NT / 2};
     if (!fp_tensor_map(&tmA, a.A, 2, da, sa, ba) || !fp_tensor_map(&tmW, a.W, 2, dw, sw, bw)) return ZKDS_ERR_UNSUPPORTED;
     const size_t smem = (size_t)stage_bytes * p.stages + kEpiWarps * kStageBlock + 1024;
-    ZKDS_CUDA(cudaFuncSetAttribute(linear_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    // always the same limit, not this launch's size: earlier launches may sit in a captured graph
+    ZKDS_CUDA(cudaFuncSetAttribute(linear_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kLinearSmemMax));
     const int tiles = few * p.ksplit;
     const unsigned grid = 2u * (unsigned)(tiles < pairs ? tiles : pairs);
     linear_tc_kernel<<<grid, kThreadsTc, smem, st>>>(tmA, tmW, p);

@@ -254,6 +254,7 @@ attention_plain_kernel(const zkfp_attention_args a)
     const long long rows = a.shared ? a.seq * a.heads : a.seq;
     const int per_tok = a.shared ? (int)a.heads : 1;
     const int start = a.start[b];
+    if (start < 0 || start + a.seq > a.base + a.keys) return;      // not a step of these keys
     const long long slot = a.slots ? a.slots[b] : b;
     const T* q = (const T*)a.q + (long long)b * a.seq * a.heads * a.q_head;
     T* out = (T*)a.out + (long long)b * a.seq * a.heads * a.o_head;
@@ -339,8 +340,9 @@ static int attention_plain(const zkfp_attention_args& a, cudaStream_t st)
 {
     const size_t smem = sizeof(float) * ((size_t)kRows * (a.d1 + a.d2 + a.dv) + kKeys * (kDimChunk + 1) + kRows * kKeys +
                                          3 * kRows);
-    if (smem > 227 * 1024) return ZKDS_ERR_UNSUPPORTED;
-    ZKDS_CUDA(cudaFuncSetAttribute(attention_plain_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    if (smem > (size_t)kSharedMax) return ZKDS_ERR_UNSUPPORTED;
+    // always the same limit: a captured launch keeps its own size, but is run under the function's current attribute
+    ZKDS_CUDA(cudaFuncSetAttribute(attention_plain_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSharedMax));
     const long long rows = a.shared ? a.seq * a.heads : a.seq;
     const dim3 grid((unsigned)((rows + kRows - 1) / kRows), a.shared ? 1u : (unsigned)a.heads, (unsigned)a.batch);
     attention_plain_kernel<T><<<grid, 256, smem, st>>>(a);

@@ -28,7 +28,7 @@ _vp, _ll, _i, _f, _d = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.
 class LinearArgs(ctypes.Structure):
     _fields_ = [("A", _vp), ("W", _vp), ("out", _vp), ("aux", _vp), ("table", _vp), ("start", _vp),
                 ("lda", _ll), ("ldw", _ll), ("ldo", _ll), ("ldaux", _ll), ("M", _ll), ("N", _ll), ("K", _ll),
-                ("seq", _ll), ("dtype", _i), ("out_dtype", _i), ("epilogue", _i), ("pairs", _i), ("period", _i),
+                ("seq", _ll), ("positions", _ll), ("dtype", _i), ("out_dtype", _i), ("epilogue", _i), ("pairs", _i), ("period", _i),
                 ("offset", _i)]
 
 
@@ -133,7 +133,7 @@ def linear(A, W, out, epilogue=STORE, aux=None, table=None, start=None, seq=1, p
     """out = epilogue(A W^T); A [M, K], W [N, K], out [M, N] (N / 2 columns with GLU)"""
     a = LinearArgs(A.data_ptr(), W.data_ptr(), out.data_ptr(), ptr(aux), ptr(table), ptr(start), A.stride(0),
                    W.stride(0), out.stride(0), aux.stride(0) if aux is not None else 0, A.shape[0], W.shape[0],
-                   W.shape[1], seq, code(A.dtype), code(out.dtype), epilogue, pairs, period, offset)
+                   W.shape[1], seq, table.shape[0] if table is not None else 0, code(A.dtype), code(out.dtype), epilogue, pairs, period, offset)
     _check(_linear(ctypes.byref(a), _stream()), "linear %dx%dx%d" % (A.shape[0], W.shape[0], W.shape[1]))
     return out
 

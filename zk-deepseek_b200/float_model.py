@@ -32,8 +32,6 @@ except ImportError:  # pragma: no cover - this directory first on sys.path
 ABSORB_MAX_TOKENS = 16
 # a step with more rows than this is run in portions (bounds the activations and the expanded keys and values)
 MAX_STEP_TOKENS = 8192
-# one-token steps are captured in a CUDA graph and replayed
-DECODE_GRAPHS = True
 
 
 def _padded(t, shape, dtype, device):
@@ -53,12 +51,12 @@ def rotary_table(rot, positions, device):
 class Step:
     """what the layers need to know about the step that is running"""
 
-    def __init__(self, batch, seq, start_pos, start, slots, host_slots, cache, bound):
+    def __init__(self, batch, seq, start_pos, start, slots, host_slots, cache):
         self.batch, self.seq, self.rows = batch, seq, batch * seq
-        self.start_pos = start_pos        # host value, None inside a captured graph
+        self.start_pos = start_pos
         self.start, self.slots = start, slots          # device int32 [batch]
         self.host_slots, self.cache = host_slots, cache
-        self.bound = bound                # most keys any query of this step could see
+        self.bound = start_pos + seq      # most keys any query of this step could see
 
 
 class RMSNorm(nn.Module):
@@ -266,7 +264,6 @@ class FloatTransformer(nn.Module):
         self.norm = RMSNorm(args.dim, args.eps)
         self.register_buffer("embed", None)
         self.cache = None
-        self._graphs = {}
         self._tables = {}
 
     # -- weights and cache --------------------------------------------------------------------------
@@ -314,7 +311,7 @@ class FloatTransformer(nn.Module):
         for s in slots:
             self.cache.extend(s, start_pos, S)
         meta = torch.tensor([[start_pos] * B, list(slots)], dtype=torch.int32).to(self.device, non_blocking=True)
-        st = Step(B, S, start_pos, meta[0], meta[1], list(slots), self.cache, start_pos + S)
+        st = Step(B, S, start_pos, meta[0], meta[1], list(slots), self.cache)
         return self._embed(tokens.to(self.device)), st
 
     def _embed(self, tokens):
@@ -347,9 +344,6 @@ class FloatTransformer(nn.Module):
         """
         B, S = tokens.shape
         info = {}
-        if S == 1 and DECODE_GRAPHS and not layer_probe and layers_out is None and (want is None or len(want)):
-            logits = self._graph_step(tokens, start_pos, slots)
-            return (logits if want is None else logits[list(want)]), info
         limit = max(ABSORB_MAX_TOKENS + 1, MAX_STEP_TOKENS // B)
         if S > limit and layers_out is None and not layer_probe:
             out = []
@@ -381,57 +375,3 @@ class FloatTransformer(nn.Module):
                 return torch.empty(0, self.args.vocab_size, device=self.device), info
             want = torch.tensor(list(want), dtype=torch.int32).to(self.device, non_blocking=True)
         return self.finish_inference(h, st, want), info
-
-    def _graph_step(self, tokens, start_pos, slots):
-        B = tokens.shape[0]
-        for s in slots:
-            self.cache.extend(s, start_pos, 1)
-        g = self._graphs.get(B)
-        if g is None:
-            g = self._graphs[B] = _DecodeGraph(self, B)
-        return g.run(tokens, start_pos, slots)
-
-
-class _DecodeGraph:
-    """The kernels of a one-token step of B sequences, captured once; tokens, positions and slots are device
-    inputs of the graph."""
-
-    def __init__(self, model, B):
-        self.model, dev = model, model.device
-        self.tokens = torch.zeros(B, 1, dtype=torch.int64, device=dev)
-        self.meta = torch.zeros(2, B, dtype=torch.int32, device=dev)
-        self.host = torch.zeros(2, B, dtype=torch.int32).pin_memory()
-        # the warm-up below runs on zero inputs: slot 0, position 0 are written with the latents of token 0, so
-        # their content is put back afterwards
-        self.st = Step(B, 1, None, self.meta[0], self.meta[1], None, model.cache, model.args.max_seq_len)
-        saved = [None if b is None else b[0, 0].clone() for b in model.cache.buffers]
-        side = torch.cuda.Stream(device=dev)
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            self._body()
-            side.synchronize()
-            self.graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(self.graph, stream=side):
-                self.logits = self._body()
-            for b, s in zip(model.cache.buffers, saved):
-                if b is not None:
-                    b[0, 0].copy_(s)
-        torch.cuda.current_stream().wait_stream(side)
-        self.copied = torch.cuda.Event()
-
-    def _body(self):
-        m = self.model
-        h = m._embed(self.tokens)
-        for layer in m.layers:
-            layer(h[0], h[1], self.st)
-        return m.finish_inference(h, self.st)
-
-    def run(self, tokens, start_pos, slots):
-        self.copied.synchronize()         # the previous step's inputs have left the pinned buffer
-        self.host[0].fill_(start_pos)
-        self.host[1].copy_(torch.tensor(slots, dtype=torch.int32))
-        self.meta.copy_(self.host, non_blocking=True)
-        self.tokens.copy_(tokens, non_blocking=True)
-        self.copied.record()
-        self.graph.replay()
-        return self.logits.clone()
