@@ -1581,9 +1581,10 @@ class FloatDesignWorkload:
     # ---- per-kernel fractions ----------------------------------------------------------------------------
     OPS = ("linear", "attention", "perhead", "latent_post", "add_norm")
 
-    def float_classes(self, model, step, seq, start, peaks, decode):
+    def float_classes(self, model, step, seq, start, peaks):
         """kernel class -> (seconds, fraction of its roofline) of one step"""
         torch, out = self.torch, {}
+        # the per-layer interface, not the recorded step, so that the timed functions are called
         with OpTimer(torch, (self.fk, self.OPS)) as timer:
             calls = timer.run(step)
         vis = self.visible(seq, start)
@@ -1688,7 +1689,7 @@ class FloatDesignWorkload:
             sec = _timed_steps(torch, _Step(lambda: self.prefill(model, self.toks, logits=False)), 10)
             row["prefill_us_per_layer"] = round(sec / n * 1e6, 1)
             row["prefill_kernels_of_%d_layers" % n] = self.float_classes(
-                model, lambda: self.prefill(model, self.toks, logits=False), self.T, 0, peaks, False)
+                model, lambda: self.prefill(model, self.toks, logits=False), self.T, 0, peaks)
             slots = model.begin_batch(1)
             model.step(self.toks, 0, slots, want=[])
             one = self.toks[:, :1]
@@ -1696,12 +1697,16 @@ class FloatDesignWorkload:
             def decode():
                 model.step(one, self.T, slots)
                 model.cache.truncate(slots[0], self.T)
+
+            def decode_layers():
+                model.step(one, self.T, slots, layers_out=[])
+                model.cache.truncate(slots[0], self.T)
             sec = _timed_steps(torch, _Step(decode), 30)
             row["decode_us_per_step"] = round(sec * 1e6, 1)
             row["decode_tokens_per_s"] = round(1 / sec, 1)
             nbytes = 2.0 * sum(b.numel() for b in model.buffers() if b is not None and b.dtype == torch.bfloat16)
             row["decode_frac_of_hbm"] = round(nbytes / (peaks["hbm_gbs"] * 1e9) / sec, 3)
-            row["decode_kernels_of_%d_layers" % n] = self.float_classes(model, decode, 1, self.T, peaks, True)
+            row["decode_kernels_of_%d_layers" % n] = self.float_classes(model, decode_layers, 1, self.T, peaks)
             model.end_batch(slots)
             if size == self.size:
                 self.model = None

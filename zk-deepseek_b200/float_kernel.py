@@ -98,6 +98,38 @@ def device_status(sync=False):
     _check(lib.zkfp_device_status(), "device status")
 
 
+class Recording:
+    """Calls made while recording, with their argument structures and the tensors they point to, to be issued again
+    without rebuilding anything: the host side of a one-token step is a loop over prepared calls."""
+
+    active = None
+
+    def __init__(self):
+        self.calls, self.held = [], []
+
+    def __enter__(self):
+        Recording.active = self
+        return self
+
+    def __exit__(self, *exc):
+        Recording.active = None
+        return False
+
+    def replay(self):
+        st = _stream()
+        for fn, args, what in self.calls:
+            rc = fn(*args, st)
+            if rc:
+                _check(rc, what)
+
+
+def _call(fn, args, what, *tensors):
+    _check(fn(*args, _stream()), what)
+    if Recording.active is not None:
+        Recording.active.calls.append((fn, args, what))
+        Recording.active.held.extend(tensors)
+
+
 def code(dtype):
     return BF16 if dtype == torch.bfloat16 else F32
 
@@ -112,34 +144,34 @@ def ptr(t):
 
 def embed(tokens, table, vocab, x, xb):
     """x [rows, pitch] = table[tokens] in 32-bit, xb the same in bfloat16 (None in float32 mode)"""
-    _check(_embed(tokens.data_ptr(), table.data_ptr(), table.stride(0), vocab, x.data_ptr(), ptr(xb), x.stride(0),
-                  x.shape[0], code(table.dtype), _stream()), "embed")
+    _call(_embed, (tokens.data_ptr(), table.data_ptr(), table.stride(0), vocab, x.data_ptr(), ptr(xb), x.stride(0),
+                   x.shape[0], code(table.dtype)), "embed", tokens, table, x, xb)
 
 
 def add_norm(x, y, w, xb, width, eps):
     """x += w * y / rms(y); xb = bfloat16(x)"""
-    _check(_add_norm(x.data_ptr(), y.data_ptr(), w.data_ptr(), ptr(xb), x.stride(0), y.stride(0), x.shape[0], width,
-                     eps, _stream()), "add_norm")
+    _call(_add_norm, (x.data_ptr(), y.data_ptr(), w.data_ptr(), ptr(xb), x.stride(0), y.stride(0), x.shape[0], width,
+                      eps), "add_norm", x, y, w, xb)
 
 
 def norm_rows(x, index, w, out, width, eps):
     """out[i] = w * x[index[i]] / rms(x[index[i]]); index None takes every row"""
-    n = out.shape[0]
-    _check(_norm_rows(x.data_ptr(), x.stride(0), ptr(index), w.data_ptr(), out.data_ptr(), out.stride(0), n, width,
-                      eps, code(out.dtype), _stream()), "norm_rows")
+    _call(_norm_rows, (x.data_ptr(), x.stride(0), ptr(index), w.data_ptr(), out.data_ptr(), out.stride(0), out.shape[0],
+                       width, eps, code(out.dtype)), "norm_rows", x, index, w, out)
 
 
 def linear(A, W, out, epilogue=STORE, aux=None, table=None, start=None, seq=1, pairs=0, period=0, offset=0):
     """out = epilogue(A W^T); A [M, K], W [N, K], out [M, N] (N / 2 columns with GLU)"""
     a = LinearArgs(A.data_ptr(), W.data_ptr(), out.data_ptr(), ptr(aux), ptr(table), ptr(start), A.stride(0),
                    W.stride(0), out.stride(0), aux.stride(0) if aux is not None else 0, A.shape[0], W.shape[0],
-                   W.shape[1], seq, table.shape[0] if table is not None else 0, code(A.dtype), code(out.dtype), epilogue, pairs, period, offset)
-    _check(_linear(ctypes.byref(a), _stream()), "linear %dx%dx%d" % (A.shape[0], W.shape[0], W.shape[1]))
+                   W.shape[1], seq, table.shape[0] if table is not None else 0, code(A.dtype), code(out.dtype),
+                   epilogue, pairs, period, offset)
+    _call(_linear, (ctypes.byref(a),), "linear", A, W, out, aux, table, start)
     return out
 
 
-def latent_post(args):
-    _check(_latent(ctypes.byref(args), _stream()), "latent_post")
+def latent_post(args, *tensors):
+    _call(_latent, (ctypes.byref(args),), "latent_post", *tensors)
 
 
 def perhead(x, W, out, transposed, copy=(0, 0, 0)):
@@ -149,11 +181,11 @@ def perhead(x, W, out, transposed, copy=(0, 0, 0)):
     a = PerHeadArgs(x.data_ptr(), W.data_ptr(), out.data_ptr(), x.stride(0), x.stride(1), out.stride(0),
                     out.stride(1), W.stride(0), W.stride(1), x.shape[0], x.shape[1], n_out, n_in, int(transposed),
                     code(x.dtype), *copy)
-    _check(_perhead(ctypes.byref(a), _stream()), "perhead")
+    _call(_perhead, (ctypes.byref(a),), "perhead", x, W, out)
 
 
-def attention(args):
-    _check(_attention(ctypes.byref(args), _stream()), "attention")
+def attention(args, *tensors):
+    _call(_attention, (ctypes.byref(args),), "attention", *tensors)
 
 
 def attention_scratch(args):

@@ -49,14 +49,15 @@ def rotary_table(rot, positions, device):
 
 
 class Step:
-    """what the layers need to know about the step that is running"""
+    """What the layers need to know about the step that is running."""
 
     def __init__(self, batch, seq, start_pos, start, slots, host_slots, cache):
         self.batch, self.seq, self.rows = batch, seq, batch * seq
-        self.start_pos = start_pos
+        self.start_pos = start_pos        # None in a recorded step
         self.start, self.slots = start, slots          # device int32 [batch]
         self.host_slots, self.cache = host_slots, cache
-        self.bound = start_pos + seq      # most keys any query of this step could see
+        # most keys any query of this step could see
+        self.bound = start_pos + seq if start_pos is not None else cache.capacity
 
 
 class RMSNorm(nn.Module):
@@ -138,7 +139,7 @@ class LatentAttention(nn.Module):
                          self.table.data_ptr(), st.start.data_ptr(), st.slots.data_ptr(), y.stride(0), cq.stride(0),
                          st.rows, st.seq, cache.stride(0), cache.stride(1), cache.shape[1], c.q_rank, self.q,
                          c.kv_rank, self.c, self.pairs, int(self.own_kv), K.code(dt), self.eps)
-        K.latent_post(a)
+        K.latent_post(a, y, cq, cache, self.q_norm, self.kv_norm, self.table, st.start, st.slots)
         q = torch.empty(st.rows, c.heads, self.d + self.r, dtype=dt, device=dev)
         K.linear(cq, self.w_uq, q.view(st.rows, -1), K.ROTATE, table=self.table, start=st.start, seq=st.seq,
                  pairs=self.pairs, period=self.d + self.r, offset=self.d)
@@ -165,7 +166,7 @@ class LatentAttention(nn.Module):
         n = K.attention_scratch(a)
         scratch = torch.empty(n, dtype=torch.float32, device=dev) if n else None
         a.scratch = K.ptr(scratch)
-        K.attention(a)
+        K.attention(a, qa, lat, cache, scratch, st.start, st.slots)
         o = torch.empty(st.rows, H, self.v, dtype=dt, device=dev)
         K.perhead(lat, uv, o, False)
         return o
@@ -265,6 +266,7 @@ class FloatTransformer(nn.Module):
         self.register_buffer("embed", None)
         self.cache = None
         self._tables = {}
+        self._recorded = {}         # batch size -> recorded one-token step
 
     # -- weights and cache --------------------------------------------------------------------------
     def load_weights(self, W, device):
@@ -344,6 +346,9 @@ class FloatTransformer(nn.Module):
         """
         B, S = tokens.shape
         info = {}
+        if S == 1 and not layer_probe and layers_out is None and (want is None or len(want)):
+            logits = self._decode(tokens, start_pos, slots)
+            return (logits if want is None else logits[list(want)]), info
         limit = max(ABSORB_MAX_TOKENS + 1, MAX_STEP_TOKENS // B)
         if S > limit and layers_out is None and not layer_probe:
             out = []
@@ -375,3 +380,46 @@ class FloatTransformer(nn.Module):
                 return torch.empty(0, self.args.vocab_size, device=self.device), info
             want = torch.tensor(list(want), dtype=torch.int32).to(self.device, non_blocking=True)
         return self.finish_inference(h, st, want), info
+
+    def _decode(self, tokens, start_pos, slots):
+        B = tokens.shape[0]
+        for s in slots:
+            self.cache.extend(s, start_pos, 1)
+        if B not in self._recorded:
+            self._recorded[B] = RecordedStep(self, B)
+        return self._recorded[B].run(tokens, start_pos, slots)
+
+
+class RecordedStep:
+    """The kernels of a one-token step of B sequences: the first run records the calls with their buffers, later runs
+    issue them again.  Tokens, positions and slots are device inputs."""
+
+    def __init__(self, model, B):
+        dev = model.device
+        self.model, self.calls = model, None
+        self.tokens = torch.zeros(B, 1, dtype=torch.int64, device=dev)
+        self.meta = torch.zeros(2, B, dtype=torch.int32, device=dev)
+        self.host = torch.zeros(2, B, dtype=torch.int32).pin_memory()
+        self.rows = torch.arange(B, dtype=torch.int32, device=dev)
+        self.copied = torch.cuda.Event()
+
+    def run(self, tokens, start_pos, slots):
+        self.copied.synchronize()         # the previous step's inputs have left the pinned buffer
+        self.host[0].fill_(start_pos)
+        for b, s in enumerate(slots):
+            self.host[1, b] = s
+        self.meta.copy_(self.host, non_blocking=True)
+        self.tokens.copy_(tokens, non_blocking=True)
+        self.copied.record()
+        if self.calls is not None:
+            self.calls.replay()
+            return self.logits.clone()
+        m = self.model
+        st = Step(self.tokens.shape[0], 1, None, self.meta[0], self.meta[1], None, m.cache)
+        with K.Recording() as calls:
+            h = m._embed(self.tokens)
+            for layer in m.layers:
+                layer(h[0], h[1], st)
+            self.logits = m.finish_inference(h, st, self.rows)
+        self.calls = calls
+        return self.logits.clone()
