@@ -15,7 +15,7 @@ from oracle import float_oracle as fo
 
 cfgmod = importlib.import_module(PKG + ".float_config")
 registry = importlib.import_module(PKG + ".registry")
-cachemod = importlib.import_module(PKG + ".latent_cache")
+cachemod = importlib.import_module(PKG + ".sequence_cache")
 
 
 # ---- the oracle against hand-made cases ---------------------------------------------------------------------
@@ -119,10 +119,10 @@ def test_bad_configurations_are_refused(edit):
         cfgmod.parse_config(cfg)
 
 
-def test_registry_names_both_families():
+def test_registry_names_every_design():
     assert registry.architecture_of({"architecture": "Munalorn"}) == "Munalorn"
     assert registry.architecture_of({"dim": 7168, "n_layers": 2}) == registry.INTEGER_MODEL
-    assert set(registry.architectures()) == {"Munalorn", registry.INTEGER_MODEL}
+    assert set(registry.architectures()) == {"Munalorn", "Vifelix", registry.INTEGER_MODEL}
     with pytest.raises(cfgmod.ConfigError):
         registry.architecture_of({"architecture": "Else"})
 
@@ -142,7 +142,7 @@ def test_tensor_files_round_trip(tmp_path):
 
 # ---- cache slots -----------------------------------------------------------------------------------------------
 def test_cache_slots_are_handed_out_and_taken_back():
-    c = cachemod.LatentCache([16, None, 24], [0, 0, 2], 2, 10, torch.float32, "cpu")
+    c = cachemod.SequenceCache([16, None, 24], [0, 0, 2], 2, 10, torch.float32, "cpu")
     assert c.buffer(1) is c.buffer(0) and c.buffer(2).shape == (2, 10, 24) and c.bytes() == 2 * 10 * 40 * 4
     a, b = c.acquire(), c.acquire()
     assert a != b and c.free_slots() == 0
@@ -160,7 +160,7 @@ def test_cache_slots_are_handed_out_and_taken_back():
         c.release(a)
     assert c.acquire() == a and c.lengths[a] == 0
     with pytest.raises(ValueError):
-        cachemod.LatentCache([None, 16], [0, 1], 1, 4, torch.float32, "cpu")
+        cachemod.SequenceCache([None, 16], [0, 1], 1, 4, torch.float32, "cpu")
 
 
 # ---- the loops that drive a model --------------------------------------------------------------------------------

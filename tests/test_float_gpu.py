@@ -375,7 +375,7 @@ def test_large_steps_run_in_portions(models, monkeypatch):
 
 def test_a_step_must_follow_what_the_slot_holds(models):
     cfg, W, model = models("WIDE", "bfloat16")
-    cache = importlib.import_module(PKG + ".latent_cache")
+    cache = importlib.import_module(PKG + ".sequence_cache")
     slots = model.begin_batch(1)
     with pytest.raises(ValueError):
         model.step(torch.tensor([[1]]), 3, slots)

@@ -25,7 +25,8 @@ FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std
 LIBRARIES = {
     "libint64gemm.so": (["capi.cu", "fixedpoint.cu", "gemm_exact.cu", "limb_gemm.cu", "converters.cu"],
                         ["common.cuh", "kernels.h", "tcgen05.cuh", "zkds_int64.h"]),
-    "libfloatops.so": (["float_capi.cu", "float_ops.cu", "float_gemm.cu", "float_gemm_tc.cu", "float_attention.cu"],
+    "libfloatops.so": (["float_capi.cu", "float_ops.cu", "float_gemm.cu", "float_gemm_tc.cu", "float_attention.cu",
+                        "float_grouped.cu", "float_recurrent.cu", "float_scan_tc.cu"],
                        ["common.cuh", "float_common.cuh", "tcgen05.cuh", "zkds_float.h"]),
 }
 INT_LIBRARY, FLOAT_LIBRARY = "libint64gemm.so", "libfloatops.so"

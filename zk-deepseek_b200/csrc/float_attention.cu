@@ -39,9 +39,11 @@ __device__ __forceinline__ float exp2_approx(float x)
 
 struct ExpandedParams {
     bf16* out;
+    const bf16* gate;
     const int* start;
-    long long o_head;
-    int seq, heads, base, window;
+    long long o_head, o_tok, gate_tok, gate_head;
+    float out_scale;
+    int seq, heads, heads_per_kv, base, window;
     int d1, d2, dv, seg1, seg2, segv;          // segments of 64 columns
     int k_slots, v_stages;                     // ring of key segments, value tiles
     float scale_log2;                          // scale * log2(e)
@@ -99,6 +101,7 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
     const int blocks = (p.seq + 2 * kTile - 1) / (2 * kTile), group0 = (int)blockIdx.x / (blocks * kHeadGroup) * kHeadGroup;
     const int in_group = (int)blockIdx.x - group0 * blocks, width = min(kHeadGroup, p.heads - group0);
     const int head = group0 + in_group % width, t0 = (blocks - 1 - in_group / width) * 2 * kTile;
+    const int kv_head = head / p.heads_per_kv;
     const int start = p.start[0];
     const KeyTiles kt = key_tiles(p, t0, start);
     const int segq = p.seg1 + p.seg2;
@@ -151,14 +154,14 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
                     if (!(ok = mbar_wait(smem_u32(&s.k_empty[ks]), kp ^ 1u, abort_flag))) break;
                     const uint32_t bar = smem_u32(&s.k_full[ks]), dst = sK + (uint32_t)ks * kSeg;
                     mbar_expect_tx(bar, kSeg);
-                    if (c < p.seg1) tma_load_3d(dst, &tmK1, c * 64, head, y, bar);
+                    if (c < p.seg1) tma_load_3d(dst, &tmK1, c * 64, kv_head, y, bar);
                     else tma_load_2d(dst, &tmK2, (c - p.seg1) * 64, y, bar);
                     if (++ks == p.k_slots) { ks = 0; kp ^= 1u; }
                 }
                 if (!ok || !mbar_wait(smem_u32(&s.v_empty[vs]), vp ^ 1u, abort_flag)) break;
                 const uint32_t bar = smem_u32(&s.v_full[vs]), dst = sV + (uint32_t)vs * bytesV;
                 mbar_expect_tx(bar, bytesV);
-                for (int c = 0; c < p.segv; ++c) tma_load_3d(dst + c * kSeg, &tmV, c * 64, head, y, bar);
+                for (int c = 0; c < p.segv; ++c) tma_load_3d(dst + c * kSeg, &tmV, c * 64, kv_head, y, bar);
                 if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }
             }
         }
@@ -301,7 +304,8 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
         if (ok && first_tile <= last_tile && mbar_wait(smem_u32(&s.o_full[g]), 0, abort_flag)) {
             tc_fence_after();
             const float r = 1.0f / l;
-            bf16* o = p.out + ((long long)t * p.heads + head) * p.o_head;
+            bf16* o = p.out + (long long)t * p.o_tok + head * p.o_head;
+            const bf16* gate = p.gate ? p.gate + (long long)t * p.gate_tok + head * p.gate_head : nullptr;
             for (int c = o_begin; c < o_end; c += 8) {
                 int32_t x[8];
                 tmem_ld8(tO + (uint32_t)c, x);
@@ -310,6 +314,12 @@ attention_expanded_kernel(const __grid_constant__ CUtensorMap tmQ1, const __grid
                     float w[8];
 #pragma unroll
                     for (int k = 0; k < 8; ++k) w[k] = __int_as_float(x[k]) * r;
+                    if (gate) {
+                        float z[8];
+                        load8(gate + c, z);
+#pragma unroll
+                        for (int k = 0; k < 8; ++k) w[k] *= sigmoid_f(z[k]) * p.out_scale;
+                    }
                     store8(o + c, w);
                 }
             }
@@ -349,6 +359,9 @@ int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st)
 {
     ExpandedParams p;
     p.out = (bf16*)a.out; p.start = a.start; p.o_head = a.o_head;
+    p.o_tok = a.o_tok ? a.o_tok : a.heads * a.o_head;
+    p.gate = (const bf16*)a.gate; p.gate_tok = a.gate_tok; p.gate_head = a.gate_head; p.out_scale = a.out_scale;
+    p.heads_per_kv = a.heads_per_kv > 1 ? a.heads_per_kv : 1;
     p.seq = (int)a.seq; p.heads = (int)a.heads; p.base = (int)a.base; p.window = a.window;
     p.d1 = a.d1; p.d2 = a.d2; p.dv = a.dv;
     p.seg1 = (a.d1 + 63) / 64; p.seg2 = (a.d2 + 63) / 64; p.segv = (a.dv + 63) / 64;
@@ -362,7 +375,8 @@ int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st)
     const uint64_t ks[2] = {(uint64_t)a.k1_head * 2, (uint64_t)a.k1_tok * 2}, k2s[1] = {(uint64_t)a.k2_tok * 2};
     const uint64_t vs[2] = {(uint64_t)a.v_head * 2, (uint64_t)a.v_tok * 2};
     const uint64_t dq1[3] = {(uint64_t)a.d1, H, S}, dq2[3] = {(uint64_t)(a.d2 ? a.d2 : 8), H, S};
-    const uint64_t dk1[3] = {(uint64_t)a.d1, H, N}, dk2[2] = {(uint64_t)(a.d2 ? a.d2 : 8), N}, dv[3] = {(uint64_t)a.dv, H, N};
+    const uint64_t G = H / (uint64_t)p.heads_per_kv;
+    const uint64_t dk1[3] = {(uint64_t)a.d1, G, N}, dk2[2] = {(uint64_t)(a.d2 ? a.d2 : 8), N}, dv[3] = {(uint64_t)a.dv, G, N};
     const uint32_t b3[3] = {64, 1, kTile}, b2[2] = {64, kTile};
     const bf16* q = (const bf16*)a.q;
     if (!fp_tensor_map(&q1, q, 3, dq1, qs, b3) || !fp_tensor_map(&q2, a.d2 ? q + a.d1 : q, 3, dq2, qs, b3) ||

@@ -64,10 +64,15 @@ static bool linear_ok(const zkfp_linear_args* a)
     if ((a->N & 7) || (a->K & 7) || (a->lda & 7) || (a->ldw & 7) || (a->ldo & 7)) return false;
     if (a->lda < a->K || a->ldw < a->K || a->M > 0x7fffffffll || a->N > 0x7fffffffll || a->K > 0x7fffffffll) return false;
     if ((uintptr_t)a->A & 15 || (uintptr_t)a->W & 15 || (uintptr_t)a->out & 15) return false;
-    if (a->epilogue != ZKFP_EPI_GLU && a->ldo < a->N) return false;
+    if (a->out2 && (a->epilogue == ZKFP_EPI_GLU || a->epilogue == ZKFP_EPI_GATE || a->split <= 0 || a->split >= a->N || (a->split & 31) ||
+                    a->ldo2 < a->N - a->split || (a->ldo2 & 7) || ((uintptr_t)a->out2 & 15)))
+        return false;
+    if ((uintptr_t)a->bias & 15) return false;
+    if (a->epilogue != ZKFP_EPI_GLU && a->ldo < (a->out2 ? a->split : a->N)) return false;
     if (a->epilogue == ZKFP_EPI_GLU && ((a->N & 15) || a->ldo < a->N / 2)) return false;
     if (a->epilogue == ZKFP_EPI_ROTATE &&
-        (!a->table || !a->start || a->seq <= 0 || a->positions <= 0 || a->positions > 0x7fffffffll || a->period <= 0 || (a->period & 1) || (a->offset & 1)))
+        (!a->table || !a->start || a->seq <= 0 || a->positions <= 0 || a->positions > 0x7fffffffll || a->period <= 0 || (a->period & 1) || (a->offset & 1) ||
+         a->rot_begin < 0 || (a->rot_begin & 1) || (a->rot_end & 1) || a->rot_end > a->N))
         return false;
     if (a->epilogue == ZKFP_EPI_GATE && (!a->aux || (a->ldaux & 7) || ((uintptr_t)a->aux & 15))) return false;
     return a->epilogue >= 0 && a->epilogue <= ZKFP_EPI_GLU && (a->dtype | a->out_dtype) <= 1;
@@ -77,7 +82,10 @@ static bool attention_ok(const zkfp_attention_args* a)
 {
     return a && a->q && a->k1 && a->k2 && a->v && a->out && a->start && a->batch > 0 && a->batch < 65536 && a->seq >= 0 &&
            a->heads > 0 && a->heads < 65536 && a->d1 > 0 && a->d2 >= 0 && a->dv > 0 && !(a->d1 & 7) && !(a->d2 & 7) &&
-           !(a->dv & 7) && a->q_head >= a->d1 + a->d2 && a->o_head >= a->dv && (a->shared || a->batch == 1);
+           !(a->dv & 7) && a->q_head >= a->d1 + a->d2 && a->o_head >= a->dv && (a->shared || a->batch == 1) && a->heads_per_kv >= 0 &&
+           (a->heads_per_kv <= 1 || (!a->shared && a->heads % a->heads_per_kv == 0)) &&
+           (!a->gate || (!a->shared && !((a->gate_tok | a->gate_head) & 7) && !((uintptr_t)a->gate & 15))) &&
+           (!a->o_tok || (!a->shared && a->o_tok >= a->heads * a->o_head && !(a->o_tok & 7)));
 }
 
 }  // namespace zkds
@@ -101,6 +109,8 @@ int zkfp_linear(const zkfp_linear_args* a, void* stream)
     e.ldo = a->ldo; e.ldaux = a->ldaux; e.seq = a->seq > 0 ? a->seq : 1; e.positions = a->positions;
     e.kind = a->epilogue; e.out_bf16 = a->out_dtype; e.aux_bf16 = a->dtype;
     e.pairs = a->pairs; e.period = a->period > 0 ? a->period : 1; e.offset = a->offset;
+    e.rot_begin = a->rot_begin; e.rot_end = a->rot_end > 0 ? a->rot_end : (int)a->N;
+    e.bias = a->bias; e.out2 = a->out2; e.ldo2 = a->ldo2; e.split = a->out2 ? a->split : a->N;
     cudaStream_t st = (cudaStream_t)stream;
     switch (zkfp_linear_path(a)) {
     case 2: return launch_linear_stream(*a, e, st);

@@ -86,6 +86,7 @@ __device__ __forceinline__ float block_sum(float v, float* red)
 }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ---- epilogues of the linear layers ------------------------------------------------------------------
 struct LinEpi {
@@ -95,7 +96,10 @@ struct LinEpi {
     const int* start;
     long long ldo, ldaux, seq, positions;
     int kind, out_bf16, aux_bf16;
-    int pairs, period, offset;
+    int pairs, period, offset, rot_begin, rot_end;
+    const float* bias;
+    float* out2;
+    long long ldo2, split;          // split: past the last column when there is no second output
 };
 
 __device__ __forceinline__ float aux_at(const LinEpi& e, long long m, long long n)
@@ -112,7 +116,8 @@ __device__ __forceinline__ int epi_position(const LinEpi& e, long long m)
 // the pair at columns (n, n + 1), n even, of the row at position pos
 __device__ __forceinline__ void rotate_pair(const LinEpi& e, int pos, int n, float& u, float& v)
 {
-    const int w = n % e.period - e.offset;
+    if (n < e.rot_begin || n >= e.rot_end) return;
+    const int w = (n - e.rot_begin) % e.period - e.offset;
     if (w < 0 || (w >> 1) >= e.pairs || (unsigned)pos >= (unsigned)e.positions) return;
     const float2 cs = e.table[(long long)pos * e.pairs + (w >> 1)];
     const float a = u * cs.x - v * cs.y;
@@ -123,6 +128,16 @@ __device__ __forceinline__ void rotate_pair(const LinEpi& e, int pos, int n, flo
 // eight finished accumulators of row m at columns n .. n + 7 (n a multiple of 8)
 __device__ __forceinline__ void epilogue8(const LinEpi& e, int pos, long long m, long long n, float (&v)[8])
 {
+    if (e.bias) {
+        float b[8];
+        load8(e.bias + n, b);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] += b[i];
+    }
+    if (n >= e.split) {
+        store8(e.out2 + m * e.ldo2 + (n - e.split), v);
+        return;
+    }
     if (e.kind == ZKFP_EPI_ROTATE) {
 #pragma unroll
         for (int i = 0; i < 8; i += 2) rotate_pair(e, pos, (int)n + i, v[i], v[i + 1]);
@@ -155,5 +170,8 @@ int launch_attention_prefill_tc(const zkfp_attention_args& a, cudaStream_t st);
 bool attention_decode_tc_takes(const zkfp_attention_args& a);
 int launch_attention_decode_tc(const zkfp_attention_args& a, cudaStream_t st);
 long long attention_decode_scratch(const zkfp_attention_args& a);
+bool scan_tc_takes(const zkfp_scan_args& a);
+int launch_scan_tc(const zkfp_scan_args& a, cudaStream_t st);
+long long scan_tc_scratch(const zkfp_scan_args& a);
 
 }  // namespace zkds

@@ -83,8 +83,29 @@ __device__ __forceinline__ void epilogue_block(const TcParams& p, float (&v)[32]
     const LinEpi& e = p.e;
     const int rows_ok = min(p.M - m0, 32), cols_ok = min(p.N - n, 32);
     if (rows_ok <= 0 || cols_ok <= 0) return;
+    if (e.bias) {
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            if (q * 8 < cols_ok) {
+                float b[8];
+                load8(e.bias + n + q * 8, b);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) v[q * 8 + i] += b[i];
+            }
+        }
+    }
+    if (n >= e.split) {                      // the split is a multiple of 32: whole blocks
+#pragma unroll
+        for (int q = 0; q < 8; ++q)
+            *reinterpret_cast<float4*>(stage + piece_at<8>(lane, q)) = make_float4(v[q * 4], v[q * 4 + 1], v[q * 4 + 2], v[q * 4 + 3]);
+        __syncwarp();
+        move_block<8, false>(stage, (uint8_t*)(e.out2 + (long long)m0 * e.ldo2 + (n - e.split)), e.ldo2 * 4, rows_ok, cols_ok / 4,
+                             lane);
+        __syncwarp();
+        return;
+    }
     if (e.kind == ZKFP_EPI_ROTATE) {
-        if (lane < rows_ok) {
+        if (lane < rows_ok && n < e.rot_end && n + 32 > e.rot_begin) {
 #pragma unroll
             for (int i = 0; i < 32; i += 2) rotate_pair(e, pos, n + i, v[i], v[i + 1]);
         }

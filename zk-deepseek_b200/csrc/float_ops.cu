@@ -10,13 +10,15 @@ namespace {
 template <typename T>
 __global__ void __launch_bounds__(256)
 embed_kernel(const long long* __restrict__ tokens, const T* __restrict__ table, long long ld_table, long long vocab,
-             float* __restrict__ x, bf16* __restrict__ xb, long long ldx)
+             float* __restrict__ x, bf16* __restrict__ xb, long long ldx, float scale)
 {
     const long long r = blockIdx.x, t = tokens[r];
     const bool ok = t >= 0 && t < vocab;
     for (long long c = threadIdx.x * 8; c < ldx; c += 256 * 8) {
         float v[8] = {};
         if (ok) load8(table + t * ld_table + c, v);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] *= scale;
         store8(x + r * ldx + c, v);
         if (xb) store8(xb + r * ldx + c, v);
     }
@@ -30,15 +32,19 @@ __device__ __forceinline__ float sum_squares8(const float (&v)[8])
     return s;
 }
 
-// one block per row; the second pass finds the row in L1 / L2
+// x += w * y / rms(y), then h = x or, with w2, h = w2 * x / rms(x): one block per row; what does not fit the registers
+// is found again in L1 / L2
+template <typename T>
 __global__ void __launch_bounds__(256)
-add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, bf16* __restrict__ xb,
-                long long ldx, long long ldy, int width, int padded, float eps)
+add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w,
+                const float* __restrict__ w2, T* __restrict__ h, long long ldx, long long ldy, int width, int padded,
+                float eps)
 {
     __shared__ float red[8];
     const long long r = blockIdx.x;
     float* xr = x + r * ldx;
     const float* yr = y + r * ldy;
+    T* hr = h + r * ldx;
     constexpr int KEEP = 4;               // 8192 values stay in registers
     float keep[KEEP][8];
     float s = 0.f;
@@ -57,14 +63,16 @@ add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float*
     }
     s = block_sum(s, red);
     const float rs = 1.0f / sqrtf(s / (float)width + eps);
-    auto apply = [&](int c, const float (&v)[8]) {
+    s = 0.f;
+    auto apply = [&](int c, float (&v)[8]) {          // leaves the new x in v
         float a[8], g[8];
         load8(xr + c, a);
         load8(w + c, g);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) a[i] += v[i] * rs * g[i];
-        store8(xr + c, a);
-        if (xb) store8(xb + r * ldx + c, a);
+        for (int i = 0; i < 8; ++i) v[i] = a[i] + v[i] * rs * g[i];
+        store8(xr + c, v);
+        if (w2) s += sum_squares8(v);
+        else if (h) store8(hr + c, v);
     };
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
@@ -75,6 +83,26 @@ add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float*
         float v[8];
         load8(yr + c, v);
         apply(c, v);
+    }
+    if (!w2) return;
+    s = block_sum(s, red);
+    const float rx = 1.0f / sqrtf(s / (float)width + eps);
+    auto write = [&](int c, const float (&v)[8]) {
+        float g[8];
+        load8(w2 + c, g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) g[i] *= v[i] * rx;
+        store8(hr + c, g);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * 256 + threadIdx.x) * 8;
+        if (c < padded) write(c, keep[k]);
+    }
+    for (int c = (KEEP * 256 + threadIdx.x) * 8; c < padded; c += 256 * 8) {
+        float v[8];
+        load8(xr + c, v);                 // written by this thread above
+        write(c, v);
     }
 }
 
@@ -250,6 +278,7 @@ attention_plain_kernel(const zkfp_attention_args a)
     float* mrow = alpha + kRows;
     float* lrow = mrow + kRows;
     const int b = blockIdx.z, head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int kv_head = a.heads_per_kv > 1 ? head / a.heads_per_kv : head;
     const long long row0 = (long long)blockIdx.x * kRows;
     const long long rows = a.shared ? a.seq * a.heads : a.seq;
     const int per_tok = a.shared ? (int)a.heads : 1;
@@ -258,9 +287,9 @@ attention_plain_kernel(const zkfp_attention_args a)
     const long long slot = a.slots ? a.slots[b] : b;
     const T* q = (const T*)a.q + (long long)b * a.seq * a.heads * a.q_head;
     T* out = (T*)a.out + (long long)b * a.seq * a.heads * a.o_head;
-    const T* k1 = (const T*)a.k1 + slot * a.slot_stride + (a.shared ? 0 : head * a.k1_head);
+    const T* k1 = (const T*)a.k1 + slot * a.slot_stride + (a.shared ? 0 : kv_head * a.k1_head);
     const T* k2 = (const T*)a.k2 + slot * a.slot_stride;
-    const T* v = (const T*)a.v + slot * a.slot_stride + (a.shared ? 0 : head * a.v_head);
+    const T* v = (const T*)a.v + slot * a.slot_stride + (a.shared ? 0 : kv_head * a.v_head);
     const int nrow = (int)(rows - row0 < kRows ? rows - row0 : kRows);
     auto flat = [&](int i) { return a.shared ? row0 + i : (row0 + i) * a.heads + head; };   // (token, head) pair
     for (int i = threadIdx.x; i < kRows * dk; i += 256) {
@@ -329,7 +358,10 @@ attention_plain_kernel(const zkfp_attention_args a)
     }
     for (int i = threadIdx.x; i < nrow * a.dv; i += 256) {
         const int rr = i / a.dv, d = i - rr * a.dv;
-        out[flat(rr) * a.o_head + d] = from_f32<T>(O[i] / lrow[rr]);
+        float o = O[i] / lrow[rr];
+        if (a.gate) o *= sigmoid_f(to_f32(((const T*)a.gate)[(row0 + rr) * a.gate_tok + head * a.gate_head + d])) * a.out_scale;
+        if (a.o_tok) out[(row0 + rr) * a.o_tok + head * a.o_head + d] = from_f32<T>(o);
+        else out[flat(rr) * a.o_head + d] = from_f32<T>(o);
     }
 }
 
@@ -361,25 +393,28 @@ using namespace zkds;
 extern "C" {
 
 int zkfp_embed(const long long* tokens, const void* table, long long ld_table, long long vocab, float* x, void* xb,
-               long long ldx, long long rows, int dtype, void* stream)
+               long long ldx, long long rows, float scale, int dtype, void* stream)
 {
     if (!tokens || !table || !x || rows < 0 || (ldx & 7) || ld_table < ldx) return ZKDS_ERR_ARG;
     if (rows == 0) return ZKDS_OK;
     cudaStream_t st = (cudaStream_t)stream;
     if (dtype == ZKFP_BF16)
-        embed_kernel<bf16><<<(unsigned)rows, 256, 0, st>>>(tokens, (const bf16*)table, ld_table, vocab, x, (bf16*)xb, ldx);
+        embed_kernel<bf16><<<(unsigned)rows, 256, 0, st>>>(tokens, (const bf16*)table, ld_table, vocab, x, (bf16*)xb, ldx, scale);
     else
-        embed_kernel<float><<<(unsigned)rows, 256, 0, st>>>(tokens, (const float*)table, ld_table, vocab, x, (bf16*)xb, ldx);
+        embed_kernel<float><<<(unsigned)rows, 256, 0, st>>>(tokens, (const float*)table, ld_table, vocab, x, (bf16*)xb, ldx, scale);
     return fp_launched();
 }
 
-int zkfp_add_norm(float* x, const float* y, const float* w, void* xb, long long ldx, long long ldy, long long rows,
-                  long long width, double eps, void* stream)
+int zkfp_add_norm(float* x, const float* y, const float* w, const float* w2, void* h, long long ldx, long long ldy,
+                  long long rows, long long width, double eps, int h_dtype, void* stream)
 {
-    if (!x || !y || !w || rows < 0 || width <= 0 || (ldx & 7) || (ldy & 7) || ldy < ldx || ldx < width) return ZKDS_ERR_ARG;
+    if (!x || !y || !w || (w2 && !h) || rows < 0 || width <= 0 || (ldx & 7) || (ldy & 7) || ldy < ldx || ldx < width) return ZKDS_ERR_ARG;
     if (rows == 0) return ZKDS_OK;
-    add_norm_kernel<<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, y, w, (bf16*)xb, ldx, ldy, (int)width, (int)ldx,
-                                                                     (float)eps);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (h_dtype == ZKFP_BF16)
+        add_norm_kernel<bf16><<<(unsigned)rows, 256, 0, st>>>(x, y, w, w2, (bf16*)h, ldx, ldy, (int)width, (int)ldx, (float)eps);
+    else
+        add_norm_kernel<float><<<(unsigned)rows, 256, 0, st>>>(x, y, w, w2, (float*)h, ldx, ldy, (int)width, (int)ldx, (float)eps);
     return fp_launched();
 }
 
