@@ -114,7 +114,7 @@ def test_scan_with_extreme_decays(K, dtype, decay):
     path, got, state, want, ws = run_scan(K, dtype, [3], 200, 2, 1, 64, 64, False, False, decay=[decay, 0.99])
     assert np.isfinite(got).all() and close(got, want, dtype)
     # steps so large that everything before a token is forgotten, beside a head that forgets nothing
-    path, got, state, want, ws = run_scan(K, dtype, [3], 200, 2, 1, 64, 64, True, False, decay=[decay * 1e4, 0.0])
+    path, got, state, want, ws = run_scan(K, dtype, [3], 200, 2, 1, 64, 64, True, False, decay=[decay * 100, 0.0])
     assert np.isfinite(got).all() and close(got, want, dtype)
 
 
