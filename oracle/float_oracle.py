@@ -160,6 +160,12 @@ def softplus(z):
     return np.logaddexp(0.0, z)
 
 
+def gated_norm(o, z, w, groups, eps):
+    """the gated row, each of its equal parts at unit root mean square, weighted"""
+    y = (o * silu(z)).reshape(len(o), groups, -1)
+    return rms_norm(y, 1.0, eps).reshape(o.shape) * w
+
+
 def mamba2(h, W, p, mx, eps, rnd=exact):
     T, H, P, N, G = len(h), mx["heads"], mx["vdim"], mx["state"], mx["groups"]
     inner = H * P
@@ -174,10 +180,7 @@ def mamba2(h, W, p, mx, eps, rnd=exact):
         g = j // (H // G)
         decay = np.exp(-np.exp(W[p + "A_log"][j]) * dt[:, j])
         o[:, j] = decayed_sums(C[:, g], B[:, g] * dt[:, j:j + 1], x[:, j], decay) + W[p + "D"][j] * x[:, j]
-    o = rnd(o.reshape(T, inner)) * silu(z)
-    parts = o.reshape(T, mx["norm_groups"], -1)
-    o = (parts / np.sqrt((parts * parts).mean(-1, keepdims=True) + eps)).reshape(T, inner) * W[p + "norm"]
-    return rnd(o) @ W[p + "o"].T
+    return rnd(gated_norm(rnd(o.reshape(T, inner)), z, W[p + "norm"], mx["norm_groups"], eps)) @ W[p + "o"].T
 
 
 def dense_ff_biased(h, W, p, rnd=exact):

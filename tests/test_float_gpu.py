@@ -17,6 +17,7 @@ from oracle import float_oracle as fo
 
 pytestmark = pytest.mark.gpu
 DTYPES = ["float32", "bfloat16"]
+CASES = ["ODD", "PEAKED", "WIDE"] + list(fc.RECURRENT)
 
 
 @pytest.fixture(scope="module")
@@ -247,7 +248,7 @@ def test_latents_reach_the_cache_normed_and_rotated(K, dtype):
 
 # ---- whole models ------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("case", ["ODD", "PEAKED", "WIDE"])
+@pytest.mark.parametrize("case", CASES)
 @pytest.mark.parametrize("n", [1, 2, 16, 17, 64, 65, 128, 129, 300])
 def test_prompt_against_the_oracle(models, case, dtype, n):
     cfg, W, model = models(case, dtype)
@@ -256,8 +257,9 @@ def test_prompt_against_the_oracle(models, case, dtype, n):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_residual_after_every_layer(models, dtype):
-    cfg, W, model = models("ODD", dtype)
+@pytest.mark.parametrize("case", ["ODD", "V_ODD", "V_WIDE"])
+def test_residual_after_every_layer(models, case, dtype):
+    cfg, W, model = models(case, dtype)
     toks, got = tokens_of(cfg, 70), []
     want = fc.Expected(cfg, W, toks)
     s = model.begin_batch(1)
@@ -269,7 +271,7 @@ def test_residual_after_every_layer(models, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("case", ["ODD", "PEAKED", "WIDE"])
+@pytest.mark.parametrize("case", CASES)
 def test_portions_and_decoding_give_the_prompt_s_logits(models, case, dtype):
     cfg, W, model = models(case, dtype)
     toks = tokens_of(cfg, 280, 7)
@@ -280,8 +282,9 @@ def test_portions_and_decoding_give_the_prompt_s_logits(models, case, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_long_decoding_past_every_window(models, dtype):
-    cfg, W, model = models("PEAKED", dtype)
+@pytest.mark.parametrize("case", ["PEAKED", "V_PEAKED"])
+def test_long_decoding_past_every_window(models, case, dtype):
+    cfg, W, model = models(case, dtype)
     toks = tokens_of(cfg, 600, 8)
     want = set(range(0, 600, 37)) | {63, 64, 65, 127, 128, 129, 192, 599}
     got = run(model, toks, [5] + [1] * 595, want)
@@ -326,9 +329,91 @@ def test_key_just_inside_and_just_outside_the_window(float_libpath, tmp_path, dt
             assert want.ok(run(model, toks.tolist(), portions), dtype)
 
 
+def key_valued_edge_model(window):
+    """One layer whose attention score between any query and the token `marker` stands out: in an unrotated direction of the
+    head every query points one way, the marker's key the same way and every other key the opposite one."""
+    cfg = fc.vifelix(40, 48, 1e-6, 2.0, [fc.parallel(4, 2, 16, 8, window, 1, 8, 8, 8, [0.9], None, scale=1.0, right_scale=0.0)])
+    W = fc.make_weights(cfg, 21)
+    W["embed"][:, 0] = 0
+    W["embed"][39, 0] = 8.0                         # only the marker has activation 0
+    for name, heads, bias in (("q", 4, 6.0), ("k", 2, -2.0)):
+        for h in range(heads):
+            W["l0.mix.left." + name][h * 16 + 15] = 0
+            W["l0.mix.left." + name + ".b"][h * 16 + 15] = bias
+    for h in range(2):
+        W["l0.mix.left.k"][h * 16 + 15, 0] = 4.0
+    W["l0.mix.left.q.norm"][15] = W["l0.mix.left.k.norm"][15] = 1.5
+    return cfg, {k: fc.bf16_round(v) for k, v in W.items()}
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_batch_equals_each_request_alone(models, dtype):
-    cfg, W, model = models("WIDE", dtype)
+@pytest.mark.parametrize("window", [2, 63, 64, 65, 127, 128, 129, 200])
+def test_key_inside_and_outside_the_window_of_key_valued_attention(float_libpath, tmp_path, dtype, window):
+    registry = importlib.import_module(PKG + ".registry")
+    cfg, W = key_valued_edge_model(window)
+    model = registry.load(fc.write_checkpoint(str(tmp_path), cfg, W), dtype=dtype, max_seq_len=512, max_batch_size=1)
+    for at in (0, 1, 60, 127, 128):
+        toks = np.random.default_rng(at).integers(0, 39, at + window + 3)
+        toks[at] = 39
+        want = fc.Expected(cfg, W, toks)
+        inside, outside = at + window - 1, at + window
+        other = toks.copy(); other[at] = 3
+        base = fc.oracle_logits(cfg, W, other)
+        assert not want.ok(base[inside:inside + 1], "bfloat16", [inside])      # the key matters inside
+        assert np.allclose(base[outside], want.logits[outside])                # and not outside
+        for portions in (None, [inside] + [1] * 4, [inside - 1, 2, 2]):
+            assert want.ok(run(model, toks.tolist(), portions), dtype)
+
+
+def memory_model(kind):
+    """One layer that writes the token `marker` into its state, hardly anything else, and reads it at every later token"""
+    if kind == "retention":
+        layer = fc.parallel(2, 1, 8, 8, 4, 2, 24, 16, 8, [0.998, 0.9995], None, left_scale=0.0)
+    else:
+        layer = fc.mamba2(2, 16, 24, 1, 4, 2)
+    cfg = fc.vifelix(40, 48, 1e-6, 2.0, [layer])
+    W = fc.make_weights(cfg, 22)
+    W["embed"][:, 0], W["embed"][:, 1] = 0, 1.0
+    W["embed"][39, 0] = 4.0                         # activation 0 is the marker's, activation 1 is everyone's
+    if kind == "retention":
+        for h in range(2):
+            for name, source in (("q", 1), ("k", 0)):
+                W["l0.mix.right." + name][h * 24:(h + 1) * 24] *= 0.05
+                W["l0.mix.right." + name][h * 24 + 20, source] = 4.0
+    else:
+        i, n = 32, 24
+        W["l0.mix.in"][2 * i:2 * i + 2 * n] *= 0.05
+        W["l0.mix.in"][2 * i + 5, 0] = 6.0          # B
+        W["l0.mix.in"][2 * i + n + 5, 1] = 6.0      # C
+        W["l0.mix.conv.b"][i:] = 0
+        W["l0.mix.conv"][i:] = np.array([0, 0, 0, 1.0])
+        W["l0.mix.A_log"][:] = (-7.0, -6.0)
+        W["l0.mix.D"][:] = 0.1
+        W["l0.mix.in"][2 * i + 2 * n:] *= 0.1
+    return cfg, {k: fc.bf16_round(v) for k, v in W.items()}
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("kind", ["retention", "mamba2"])
+def test_a_token_far_back_is_remembered(float_libpath, tmp_path, kind, dtype):
+    registry = importlib.import_module(PKG + ".registry")
+    cfg, W = memory_model(kind)
+    model = registry.load(fc.write_checkpoint(str(tmp_path), cfg, W), dtype=dtype, max_seq_len=640, max_batch_size=2)
+    for at in (0, 1, 2, 127, 128, 255):
+        toks = np.random.default_rng(at).integers(0, 39, at + 330)
+        toks[at] = 39
+        want, other = fc.Expected(cfg, W, toks), toks.copy()
+        other[at] = 3
+        last = len(toks) - 1
+        assert not want.ok(fc.oracle_logits(cfg, W, other)[last:], "bfloat16", [last])     # the token matters to the end
+        for portions in (None, [at + 1, 2], [max(at, 1), 1, 16, 17, 200], [128, 128], [at + 300] + [1] * 30, [2] * 20):
+            assert want.ok(run(model, toks.tolist(), portions), dtype), portions
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case", ["WIDE", "V_WIDE", "V_ODD"])
+def test_batch_equals_each_request_alone(models, case, dtype):
+    cfg, W, model = models(case, dtype)
     rows = [tokens_of(cfg, 150, 30 + b) for b in range(3)]
     slots = model.begin_batch(3)
     got = [[] for _ in rows]
@@ -344,8 +429,9 @@ def test_batch_equals_each_request_alone(models, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_a_used_slot_leaves_nothing_behind(models, dtype):
-    cfg, W, model = models("PEAKED", dtype)
+@pytest.mark.parametrize("case", ["PEAKED", "V_PEAKED", "V_ODD"])
+def test_a_used_slot_leaves_nothing_behind(models, case, dtype):
+    cfg, W, model = models(case, dtype)
     short = tokens_of(cfg, 40, 50)
     first = run(model, short, [20, 2] + [1] * 18)
     for seed in range(3):                            # longer requests fill the slot with other latents
@@ -355,8 +441,24 @@ def test_a_used_slot_leaves_nothing_behind(models, dtype):
     assert model.cache.free_slots() == model.cache.slots
 
 
-def test_large_steps_run_in_portions(models, monkeypatch):
-    cfg, W, model = models("WIDE", "float32")
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_requests_take_turns(models, dtype):
+    """two requests of different lengths, their portions interleaved, slots side by side"""
+    cfg, W, model = models("V_WIDE", dtype)
+    rows = [tokens_of(cfg, n, 40 + n) for n in (260, 90)]
+    slots, at, got = [model.begin_batch(1) for _ in rows], [0, 0], [[], []]
+    for r, n in ((0, 130), (1, 3), (0, 1), (1, 40), (0, 20), (1, 1), (0, 2), (1, 46), (0, 107)):
+        part = torch.tensor([rows[r][at[r]:at[r] + n]])
+        got[r].append(model.step(part, at[r], slots[r], want=list(range(n)))[0].cpu().numpy())
+        at[r] += n
+    for r in range(2):
+        assert at[r] == len(rows[r]) and fc.Expected(cfg, W, rows[r]).ok(np.concatenate(got[r]), dtype)
+        model.end_batch(slots[r])
+
+
+@pytest.mark.parametrize("case", ["WIDE", "V_WIDE"])
+def test_large_steps_run_in_portions(models, case, monkeypatch):
+    cfg, W, model = models(case, "float32")
     fm = importlib.import_module(PKG + ".float_model")
     monkeypatch.setattr(fm, "MAX_STEP_TOKENS", 100)
     rows = [tokens_of(cfg, 130, 70 + b) for b in range(2)]
@@ -397,7 +499,7 @@ def oracle_greedy(cfg, W, prompt, n):
     return toks[len(prompt):], margin
 
 
-@pytest.mark.parametrize("case", ["ODD", "PEAKED"])
+@pytest.mark.parametrize("case", ["ODD", "PEAKED", "V_ODD", "V_PEAKED"])
 def test_greedy_generation_of_unequal_prompts(models, case):
     G = importlib.import_module(PKG + ".generate")
     cfg, W, model = models(case, "float32")
@@ -417,9 +519,10 @@ def test_greedy_generation_of_unequal_prompts(models, case):
     assert len(probe[0]["layer_tokens"]) == len(cfg["layers"])
 
 
-def test_bfloat16_generation_follows_its_own_logits(models):
+@pytest.mark.parametrize("case", ["WIDE", "V_WIDE"])
+def test_bfloat16_generation_follows_its_own_logits(models, case):
     G = importlib.import_module(PKG + ".generate")
-    cfg, W, model = models("WIDE", "bfloat16")
+    cfg, W, model = models(case, "bfloat16")
     prompt = tokens_of(cfg, 140, 90)
     out = G.generate(model, [prompt], 40, eos_id=-5)[0]
     logits = run(model, prompt + out)
@@ -431,8 +534,9 @@ def test_bfloat16_generation_follows_its_own_logits(models):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_trace_and_generate_programs(float_libpath, tmp_path, dtype):
-    cfg = fc.ODD
+@pytest.mark.parametrize("case", ["ODD", "V_ODD"])
+def test_trace_and_generate_programs(float_libpath, tmp_path, case, dtype):
+    cfg = getattr(fc, case)
     W = fc.make_weights(cfg, 12)
     path = fc.write_checkpoint(str(tmp_path / "m"), cfg, W)
     out = tmp_path / "out"

@@ -161,7 +161,7 @@ def test_short_conv_in_portions(K, dtype, taps, portions):
 
 # ---- gated norm -----------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,vdim,part", [(3, 24, 24), (4, 20, 20), (6, 48, 96), (6, 48, 144), (3, 20, 30), (2, 12, 4), (4, 64, 256),
+@pytest.mark.parametrize("heads,vdim,part", [(3, 24, 24), (4, 20, 20), (6, 40, 80), (10, 24, 120), (3, 20, 30), (2, 12, 4), (4, 64, 256),
                                              (1, 8, 8), (12, 128, 1536), (5, 100, 250), (10, 100, 1000)])
 def test_gated_norm(K, dtype, heads, vdim, part):
     dt, p, rows = getattr(torch, dtype), (vdim + 7) // 8 * 8, 5
