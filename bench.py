@@ -1493,7 +1493,7 @@ class FloatDesignWorkload:
         self.fm = importlib.import_module(PKG + ".float_model")
         self.fc = importlib.import_module(PKG + ".float_config")
         self.fk = importlib.import_module(PKG + ".float_kernel")
-        self.size = "w7168_h128"
+        self.size = next(iter(self.SIZES))
         self.model = self.build(self.size, self.T)
         g = torch.Generator().manual_seed(3)
         self.tok_host = torch.randint(0, self.VOCAB, (1, self.T), generator=g).pin_memory()
@@ -1513,13 +1513,23 @@ class FloatDesignWorkload:
             if i % 2:
                 mx["kv_from"] = i - 1
             cfg["layers"].append({"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": ff}})
-        args = self.fc.parse_config(cfg)
-        args.max_seq_len, args.max_batch_size = self.T + 64, 1
+        return self.load(cfg, self.T + 64)
+
+    def load(self, cfg, positions):
+        """the model of a configuration with random weights"""
+        torch, args = self.torch, self.fc.parse_config(cfg)
+        args.max_seq_len, args.max_batch_size = positions, 1
         g = torch.Generator(device=self.dev).manual_seed(1)
+        around_zero = args.design.norm_offset != 0
 
         def weights(name, shape):
             t = torch.randn(shape, generator=g, device=self.dev, dtype=torch.bfloat16)
-            return t * 0.1 + 1 if "norm" in name else (t if name == "embed" else t * shape[1] ** -0.5)
+            if name.endswith((".A_log", ".dt_bias")):
+                return t.float() * 0.5 - 2.0
+            if len(shape) == 1:
+                zero = name.endswith(".b") or around_zero and not name.endswith((".q.norm", ".k.norm", "mix.norm", ".D"))
+                return t * 0.1 if zero else t * 0.1 + 1
+            return t if name == "embed" else t * shape[1] ** -0.5
         return self.fm.FloatTransformer(args).load_weights(weights, torch.device(self.dev))
 
     def config(self):
@@ -1587,28 +1597,30 @@ class FloatDesignWorkload:
         # the per-layer interface, not the recorded step, so that the timed functions are called
         with OpTimer(torch, (self.fk, self.OPS)) as timer:
             calls = timer.run(step)
-        vis = self.visible(seq, start)
         for name, a, sec in calls:
-            if name == "linear":
-                M, (N, Kd) = a[0].shape[0], a[1].shape
-                flops, nbytes = 2.0 * M * N * Kd, 2.0 * (N * Kd + M * (N + Kd))
-                if N == self.VOCAB:
-                    continue
-            elif name == "attention":
-                t = a[0]
-                flops = 2.0 * vis * t.heads * (t.d1 + t.d2 + t.dv)
-                nbytes = 2.0 * (start + seq) * (t.d1 + t.d2) * (1 if t.shared else t.heads) + \
-                    2.0 * seq * t.heads * (t.d1 + t.d2 + t.dv)
-            elif name == "perhead":
-                flops, nbytes = 2.0 * a[0].shape[0] * a[1].numel(), 2.0 * a[1].numel()
-            elif name == "add_norm":
-                flops, nbytes = 0.0, a[0].numel() * (4 + 4 + 4 + 2.0)
-            else:
-                flops, nbytes = 0.0, a[0].rows * (4.0 * a[0].ldy + 2 * (a[0].ldq + a[0].pitch))
+            cost = self.cost(name, a, seq, start)
+            if cost is None:
+                continue
             o = out.setdefault(name, [0.0, 0.0])
             o[0] += sec
-            o[1] += max(flops / (peaks["bf16_tflops"] * 1e12), nbytes / (peaks["hbm_gbs"] * 1e9))
+            o[1] += max(cost[0] / (peaks["bf16_tflops"] * 1e12), cost[1] / (peaks["hbm_gbs"] * 1e9))
         return {n: {"us": round(s * 1e6, 1), "frac": round(r / s, 3)} for n, (s, r) in out.items()}
+
+    def cost(self, name, a, seq, start):
+        """(operations, bytes) of a call, None for calls that are not counted"""
+        if name == "linear":
+            M, (N, Kd) = a[0].shape[0], a[1].shape
+            return None if N == self.VOCAB else (2.0 * M * N * Kd, 2.0 * (N * Kd + M * (N + Kd)))
+        if name == "attention":
+            t = a[0]
+            return (2.0 * self.visible(seq, start) * t.heads * (t.d1 + t.d2 + t.dv),
+                    2.0 * (start + seq) * (t.d1 + t.d2) * (1 if t.shared else t.heads) +
+                    2.0 * seq * t.heads * (t.d1 + t.d2 + t.dv))
+        if name == "perhead":
+            return 2.0 * a[0].shape[0] * a[1].numel(), 2.0 * a[1].numel()
+        if name == "add_norm":
+            return 0.0, a[0].numel() * (4 + 4 + 4 + 2.0)
+        return 0.0, a[0].rows * (4.0 * a[0].ldy + 2 * (a[0].ldq + a[0].pitch))
 
     @staticmethod
     def visible(seq, start):
@@ -1738,6 +1750,152 @@ class FloatDesignWorkload:
                 "traffic_note": "%d x %d x %d, source of the peak: %s" % (self.T, 2 * ff, w, peaks["source"])}
 
 
+class VifelixWorkload(FloatDesignWorkload):
+    """Vifelix, a decoder of Mamba-2 layers and layers with windowed attention beside retention, random bfloat16 weights at
+    the sizes of a real model's layers: prefill of one 4096-token prompt through one layer of each kind (the second with a
+    feed-forward) and the output projection of the last position.  `sizes` holds prefill and one-token decode at three
+    sizes, the roofline fraction of every kernel class, and the same of Munalorn at equal width, heads and feed-forward."""
+    name = "vifelix_prefill_4096"
+    metric = "vifelix_prefill_tokens_per_s"
+    #        width, attention heads, key heads, retention heads, Mamba-2 heads, ff
+    SIZES = {"w7168_h128": (7168, 128, 16, 28, 224, 18432), "w4096_h32": (4096, 32, 8, 16, 128, 14336),
+             "w2048_h16": (2048, 16, 4, 8, 64, 8192)}
+    DIM, R_DIM, R_VDIM, M_VDIM, STATE, GROUPS = 128, 128, 256, 64, 128, 8
+
+    def build(self, size, window):
+        w, H, G, R, M, ff = self.SIZES[size]
+        left = {"heads": H, "kv_heads": G, "dim": self.DIM, "mask": {"size": window}, "rot": {"base": 10000.0, "dims": self.DIM},
+                "scale": self.DIM ** -0.5}
+        right = {"heads": R, "dim": self.R_DIM, "vdim": self.R_VDIM, "decay": [1 - 2.0 ** (-5 - i % 8) for i in range(R)],
+                 "rot": {"base": 10000.0, "dims": self.R_DIM}}
+        return self.load({"architecture": "Vifelix", "vocab": self.VOCAB, "width": w, "norm": {"eps": 1e-6},
+                          "embedding": {"scale": 1.0}, "layers": [
+                              {"type": "mamba2", "mlp": None, "mixer": {
+                                  "heads": M, "vdim": self.M_VDIM, "state": self.STATE, "groups": self.GROUPS, "conv": 4,
+                                  "norm_groups": self.GROUPS}},
+                              {"type": "parallel", "mlp": {"kind": "dense", "ff": ff}, "mixer": {
+                                  "left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0}}]}, self.T + 256)
+
+    def config(self):
+        w, H, G, R, M, ff = self.SIZES[self.size]
+        return {"workload": self.name, "model": "Vifelix (random weights)", "global_batch": 1, "seq_len": self.T,
+                "layers": "mamba2, parallel + dense", "width": w, "heads": H, "kv_heads": G, "retention_heads": R,
+                "mamba2_heads": M, "ff": ff, "window": self.T, "l2": "weights streamed per step (over 2 GB) far exceed L2"}
+
+    def check(self, orc):
+        """1 if a small prompt's logits are further from the float64 oracle than bfloat16 rounding explains"""
+        import numpy as np
+        from oracle import float_oracle as fo
+        torch = self.torch
+        cfg = {"architecture": "Vifelix", "vocab": 256, "width": 160, "norm": {"eps": 1e-6}, "embedding": {"scale": 2.0}, "layers": [
+            {"type": "mamba2", "mlp": None, "mixer": {"heads": 4, "vdim": 32, "state": 64, "groups": 2, "conv": 4, "norm_groups": 2}},
+            {"type": "parallel", "mlp": {"kind": "dense", "ff": 200}, "mixer": {
+                "left": {"heads": 4, "kv_heads": 2, "dim": 48, "mask": {"size": 100}, "rot": {"base": 1e4, "dims": 48}, "scale": 0.15},
+                "right": {"heads": 3, "dim": 32, "vdim": 64, "decay": [0.9, 0.97, 0.99], "rot": {"base": 1e4, "dims": 32}},
+                "left_scale": 0.8, "right_scale": 0.9}}]}
+        args = self.fc.parse_config(cfg)
+        args.max_seq_len = 256
+        W, g = {}, torch.Generator().manual_seed(5)
+
+        def weights(name, shape):
+            t = torch.randn(shape, generator=g)
+            t = (t * (shape[1] ** -0.5 if len(shape) > 1 and name != "embed" else 0.5)).to(torch.bfloat16)
+            W[name] = t.double().numpy()
+            return t
+        model = self.fm.FloatTransformer(args).load_weights(weights, torch.device(self.dev))
+        toks = torch.randint(0, 256, (1, 200), generator=g)
+        slots = model.begin_batch(1)
+        got = torch.cat([model.step(toks[:, :150], 0, slots, want=range(150))[0]] +
+                        [model.step(toks[:, p:p + 1], p, slots)[0] for p in range(150, 200)]).double().cpu().numpy()
+        want = fo.forward(cfg, W, toks[0].tolist())
+        self.fk.device_status(sync=True)
+        return int(np.sqrt(((got - want) ** 2).mean()) > 0.03 * want.std())
+
+    OPS = ("linear", "attention", "heads_post", "grouped_attention", "short_conv", "scan", "gated_norm", "add_norm")
+
+    def cost(self, name, a, seq, start):
+        t = a[0]
+        if name == "linear":
+            return super().cost(name, a, seq, start)
+        if name == "attention":                     # keys and values of the key heads, queries, outputs and gates
+            kv = t.heads // t.heads_per_kv
+            return (2.0 * self.visible(seq, start) * t.heads * (t.d1 + t.dv),
+                    2.0 * ((start + seq) * kv * (t.d1 + t.dv) + seq * t.heads * (t.d1 + 2 * t.dv)))
+        if name == "grouped_attention":
+            return (4.0 * self.visible(seq, start) * t.heads * t.d,
+                    2.0 * ((start + seq) * t.kv_heads * 2 * t.d + seq * t.heads * 3 * t.d))
+        if name == "heads_post":
+            return 0.0, 2.0 * t.rows * t.d * (2 * t.heads + 3 * t.kv_heads)
+        if name == "short_conv":
+            return 0.0, 2.0 * t.batch * t.seq * 2 * t.channels
+        if name == "scan":                          # the recurrence itself, whatever form it is computed in
+            qk = t.heads // t.heads_per_qk * t.n
+            return (4.0 * t.batch * t.seq * t.heads * t.n * t.p,
+                    2.0 * t.batch * t.seq * (2 * qk + 2 * t.heads * t.p) + 8.0 * t.batch * t.heads * t.n * t.p)
+        if name == "gated_norm":
+            return 0.0, 2.0 * t.rows * 3 * t.heads * t.p
+        return super().cost(name, a, seq, start)
+
+    def measure(self, workload, model, peaks):
+        """prefill and decode of one model, each whole and by kernel class"""
+        torch, row = self.torch, {}
+        n = model.args.n_layers
+        whole = lambda: workload.prefill(model, self.toks, logits=False)
+        row["prefill_us"] = round(_timed_steps(torch, _Step(whole), 10) * 1e6, 1)
+        row["prefill_tokens_per_s_of_%d_layers" % n] = round(self.T / row["prefill_us"] * 1e6)
+        row["prefill_kernels"] = workload.float_classes(model, whole, self.T, 0, peaks)
+        slots = model.begin_batch(1)
+        model.step(self.toks, 0, slots, want=[])
+        one, at = self.toks[:, :1], [self.T]
+
+        def decode(**kw):                           # the sequence grows: a recurrent state cannot go back
+            model.step(one, at[0], slots, **kw)
+            at[0] += 1
+            if at[0] == model.args.max_seq_len:
+                model.end_batch(slots)
+                slots[:] = model.begin_batch(1)
+                model.step(self.toks, 0, slots, want=[])
+                at[0] = self.T
+        sec = _timed_steps(torch, _Step(decode), 30)
+        row["decode_us_per_step"], row["decode_tokens_per_s"] = round(sec * 1e6, 1), round(1 / sec, 1)
+        nbytes = 2.0 * sum(b.numel() for b in model.buffers() if b is not None and b.dtype == torch.bfloat16)
+        if not model.args.design.tied_output:
+            nbytes -= 2.0 * model.embed.numel()     # one row of it is read
+        row["decode_frac_of_hbm"] = round(nbytes / (peaks["hbm_gbs"] * 1e9) / sec, 3)
+        row["decode_kernels"] = workload.float_classes(model, lambda: decode(layers_out=[]), 1, self.T, peaks)
+        model.end_batch(slots)
+        return row
+
+    def sizes(self, peaks):
+        table = {}
+        other = FloatDesignWorkload.__new__(FloatDesignWorkload)
+        for n in ("torch", "ik", "dev", "fm", "fc", "fk"):
+            setattr(other, n, getattr(self, n))
+        for size in self.SIZES:
+            model = self.model if size == self.size else self.build(size, self.T)
+            row = self.measure(self, model, peaks)
+            self.model = model = None
+            self.torch.cuda.empty_cache()
+            model = other.build(size, self.T)
+            row["munalorn"] = other_row = self.measure(other, model, peaks)
+            other_row["layers"] = model.args.n_layers
+            model = None
+            self.torch.cuda.empty_cache()
+            table[size] = row
+        return {"sizes": table}
+
+    def roofline(self, peaks):
+        """the scan of the Mamba-2 layer"""
+        with OpTimer(self.torch, (self.fk, ("scan",))) as timer:
+            call = timer.run(lambda: self.prefill(self.model, self.toks, logits=False), 10)[0]
+        flops, nbytes = self.cost("scan", call[1], self.T, 0)
+        t = call[1][0]
+        return {"bound": "memory", "kernel": "scan_chunk_kernel and the kernel that makes its decays (Mamba-2 layer)",
+                "achieved": round(nbytes / call[2] / 1e9, 1), "peak": peaks["hbm_gbs"], "unit": "GB/s",
+                "frac": round(nbytes / call[2] / 1e9 / peaks["hbm_gbs"], 4), "kernel_us": round(call[2] * 1e6, 1),
+                "traffic_note": "%d tokens, %d heads of %d x %d, source of the peak: %s" % (self.T, t.heads, t.n, t.p, peaks["source"])}
+
+
 class _Step:
     def __init__(self, fn):
         self.step = fn
@@ -1748,7 +1906,7 @@ WORKLOADS = {"gemm": GemmWorkload, "gemm_prof": GemmProfWorkload, "gemm_cfg1": G
              "chain_prof": ChainProfWorkload, "mla": MlaWorkload, "mla_ref": MlaRefScaleWorkload,
              "mla_small": MlaSmallWorkload, "mla_causal": MlaCausalSkipWorkload, "moe": MoeWorkload,
              "moe_small": MoeSmallWorkload, "decode": DecodeWorkload, "decode_sharded": DecodeShardedWorkload,
-             "munalorn": FloatDesignWorkload}
+             "munalorn": FloatDesignWorkload, "vifelix": VifelixWorkload}
 DEFAULT_WORKLOAD = "mla"
 
 
@@ -1936,7 +2094,7 @@ def main():
                          "timed numbers are taken before it)")
     ap.add_argument("--no-extras", action="store_true",
                     help="default workload: leave out the GEMM, small-M, reference-scale and reference-kernel parts; "
-                         "munalorn: leave out the table of sizes")
+                         "munalorn, vifelix: leave out the table of sizes")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup
 

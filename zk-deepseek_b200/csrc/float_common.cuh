@@ -86,6 +86,10 @@ __device__ __forceinline__ float block_sum(float v, float* red)
 }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+// for results that are rounded to T: a few ulps of 32-bit where T is bfloat16
+template <typename T> __device__ __forceinline__ float sigmoid_for(float z);
+template <> __device__ __forceinline__ float sigmoid_for<float>(float z) { return sigmoid_f(z); }
+template <> __device__ __forceinline__ float sigmoid_for<bf16>(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ---- epilogues of the linear layers ------------------------------------------------------------------

@@ -9,7 +9,7 @@ namespace {
 // ---- short convolution -------------------------------------------------------------------------------------------
 // A thread owns eight channels of a tile of tokens.  The threads of a sequence's first tile read the inputs before the
 // step from the state, and are the ones that replace it.  TAPS 0: any number of taps, inputs read again for every tap.
-constexpr int kConvTokens = 32;
+constexpr int kConvTokens = 32, kConvBatch = 8;    // tokens of a tile, and those whose inputs are in flight together
 
 template <typename T>
 __device__ __forceinline__ void conv_input(const zkfp_conv_args& a, const T* x, const T* state, int t, int c, bool fresh,
@@ -43,22 +43,31 @@ short_conv_kernel(const zkfp_conv_args a)
         for (int j = 0; j < TAPS; ++j) load8(a.w + (long long)j * a.channels + c, w[j]);
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) conv_input(a, x, state, t0 - (TAPS - 1) + j, c, fresh, ring[j]);
-#pragma unroll 4
-        for (int t = t0; t < t1; ++t) {
-            load8(x + t * a.ldx + c, ring[TAPS - 1]);
-            float v[8];
+        for (int tb = t0; tb < t1; tb += kConvBatch) {
+            uint4 raw[kConvBatch][sizeof(T) / 2];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                v[i] = bias[i];
+            for (int k = 0; k < kConvBatch; ++k)
+                if (tb + k < t1)
 #pragma unroll
-                for (int j = 0; j < TAPS; ++j) v[i] = fmaf(w[j][i], ring[j][i], v[i]);
-                v[i] *= sigmoid_f(v[i]);
+                    for (int q = 0; q < (int)sizeof(T) / 2; ++q) raw[k][q] = reinterpret_cast<const uint4*>(x + (tb + k) * a.ldx + c)[q];
+#pragma unroll
+            for (int k = 0; k < kConvBatch; ++k) {
+                if (tb + k >= t1) break;
+                load8(reinterpret_cast<const T*>(raw[k]), ring[TAPS - 1]);
+                float v[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    v[i] = bias[i];
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) v[i] = fmaf(w[j][i], ring[j][i], v[i]);
+                    v[i] *= sigmoid_for<T>(v[i]);
+                }
+                store8(out + (tb + k) * a.ldo, v);
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) ring[j][i] = ring[j + 1][i];
             }
-            store8(out + t * a.ldo, v);
-#pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j)
-#pragma unroll
-                for (int i = 0; i < 8; ++i) ring[j][i] = ring[j + 1][i];
         }
     } else {
         for (int t = t0; t < t1; ++t) {
@@ -73,7 +82,7 @@ short_conv_kernel(const zkfp_conv_args a)
                 for (int i = 0; i < 8; ++i) v[i] = fmaf(w[i], in[i], v[i]);
             }
 #pragma unroll
-            for (int i = 0; i < 8; ++i) v[i] *= sigmoid_f(v[i]);
+            for (int i = 0; i < 8; ++i) v[i] *= sigmoid_for<T>(v[i]);
             store8(out + t * a.ldo, v);
         }
     }
@@ -203,9 +212,9 @@ int scan(const zkfp_scan_args& a, cudaStream_t st)
 }
 
 // ---- gated norm --------------------------------------------------------------------------------------------------
-// THREADS threads take one part of one row.  PACKED: parts are contiguous runs of whole 8-element vectors (`p` apart when
-// a part is a head, whose padding holds zeros); otherwise elements are addressed one by one.
-template <typename T, int THREADS, bool PACKED>
+// Parts that are contiguous runs of whole 8-element vectors (a head with its zero padding, or several whole heads without
+// any): THREADS threads take one part of one row and keep KEEP vectors each.  FIRST: the gate comes before the norm.
+template <typename T, int THREADS, int KEEP, bool FIRST>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const zkfp_gated_norm_args a, int parts, int stride)
 {
@@ -213,105 +222,126 @@ gated_norm_kernel(const zkfp_gated_norm_args a, int parts, int stride)
     const long long unit = (long long)blockIdx.x * (256 / THREADS) + threadIdx.x / THREADS;
     if (unit >= a.rows * parts) return;                  // whole warps, or the whole block
     const long long r = unit / parts;
-    const int part = (int)(unit - r * parts), lane = threadIdx.x % THREADS;
+    const int c0 = (int)(unit - r * parts) * stride, lane = threadIdx.x % THREADS;
+    const T* x = (const T*)a.x + r * a.ldx + c0;
+    const T* g = (const T*)a.g + r * a.ldg + c0;
+    T* out = (T*)a.out + r * a.ldo + c0;
+    float y[KEEP][8], z[FIRST ? 1 : KEEP][8];
+    float s = 0.f;
+    auto load = [&](int c, float (&v)[8], float (&u)[8]) {
+        load8(x + c, v);
+        load8(g + c, u);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) u[i] *= sigmoid_for<T>(u[i]);
+        if (FIRST) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] *= u[i];
+        }
+    };
+    auto add = [&](const float (&v)[8]) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s = fmaf(v[i], v[i], s);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * THREADS + lane) * 8;
+        if (c < stride) {
+            load(c, y[k], z[FIRST ? 0 : k]);
+            add(y[k]);
+        }
+    }
+    for (int c = (KEEP * THREADS + lane) * 8; c < stride; c += THREADS * 8) {
+        float v[8], u[8];
+        load(c, v, u);
+        add(v);
+    }
+    s = THREADS == 32 ? warp_sum(s) : block_sum(s, red);
+    const float rs = 1.0f / sqrtf(s / (float)a.part + (float)a.eps);
+    auto write = [&](int c, float (&v)[8], const float (&u)[8]) {
+        if (FIRST) {
+            float w[8];
+            load8(a.weight + c0 + c, w);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] *= rs * w[i];
+        } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] *= rs * u[i] * a.scale;
+        }
+        store8(out + c, v);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * THREADS + lane) * 8;
+        if (c < stride) write(c, y[k], z[FIRST ? 0 : k]);
+    }
+    for (int c = (KEEP * THREADS + lane) * 8; c < stride; c += THREADS * 8) {
+        float v[8], u[8];
+        load(c, v, u);
+        write(c, v, u);
+    }
+}
+
+// any part: a block per part of a row, elements one by one
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_norm_any_kernel(const zkfp_gated_norm_args a, int parts)
+{
+    __shared__ float red[8];
+    const long long r = blockIdx.x / parts;
+    const int part = (int)(blockIdx.x - r * parts);
     const T* x = (const T*)a.x + r * a.ldx;
     const T* g = (const T*)a.g + r * a.ldg;
     T* out = (T*)a.out + r * a.ldo;
-    const bool first = a.weight != nullptr;              // the gate comes before the norm
-    float s = 0.f;
-    auto norm = [&](float sum) {
-        sum = THREADS == 32 ? warp_sum(sum) : block_sum(sum, red);
-        return 1.0f / sqrtf(sum / (float)a.part + (float)a.eps);
+    auto at = [&](int e) {
+        const int h = e / a.vdim;
+        return h * a.p + e - h * a.vdim;
     };
-    if constexpr (PACKED) {
-        const int c0 = part * stride;
-        constexpr int KEEP = 4;
-        float y[KEEP][8], z[KEEP][8];
-        auto load = [&](int c, float (&v)[8], float (&u)[8]) {
-            load8(x + c, v);
-            load8(g + c, u);
-#pragma unroll
-            for (int i = 0; i < 8; ++i) u[i] *= sigmoid_f(u[i]);
-            if (first) {
-#pragma unroll
-                for (int i = 0; i < 8; ++i) v[i] *= u[i];
-            }
-#pragma unroll
-            for (int i = 0; i < 8; ++i) s = fmaf(v[i], v[i], s);
-        };
-#pragma unroll
-        for (int k = 0; k < KEEP; ++k) {
-            const int c = (k * THREADS + lane) * 8;
-            if (c < stride) load(c0 + c, y[k], z[k]);
-        }
-        for (int c = (KEEP * THREADS + lane) * 8; c < stride; c += THREADS * 8) {
-            float v[8], u[8];
-            load(c0 + c, v, u);
-        }
-        const float rs = norm(s);
-        auto write = [&](int c, float (&v)[8], const float (&u)[8]) {
-            if (first) {
-                float w[8];
-                load8(a.weight + c, w);
-#pragma unroll
-                for (int i = 0; i < 8; ++i) v[i] *= rs * w[i];
-            } else {
-#pragma unroll
-                for (int i = 0; i < 8; ++i) v[i] *= rs * u[i] * a.scale;
-            }
-            store8(out + c, v);
-        };
-#pragma unroll
-        for (int k = 0; k < KEEP; ++k) {
-            const int c = (k * THREADS + lane) * 8;
-            if (c < stride) write(c0 + c, y[k], z[k]);
-        }
-        for (int c = (KEEP * THREADS + lane) * 8; c < stride; c += THREADS * 8) {
-            float v[8], u[8], t = s;
-            load(c0 + c, v, u);
-            s = t;
-            write(c0 + c, v, u);
-        }
-    } else {
-        auto at = [&](int e) {
-            const int h = e / a.vdim;
-            return h * a.p + e - h * a.vdim;
-        };
-        auto gate = [&](int c) {
-            const float u = to_f32(g[c]);
-            return u * sigmoid_f(u);
-        };
-        for (int e = part * a.part + lane; e < (part + 1) * a.part; e += THREADS) {
-            const int c = at(e);
-            const float v = to_f32(x[c]) * (first ? gate(c) : 1.f);
-            s = fmaf(v, v, s);
-        }
-        const float rs = norm(s);
-        for (int e = part * a.part + lane; e < (part + 1) * a.part; e += THREADS) {
-            const int c = at(e);
-            out[c] = from_f32<T>(to_f32(x[c]) * gate(c) * rs * (first ? a.weight[c] : a.scale));
-        }
-        if (part == 0)                                   // padding of every head
-            for (int e = lane; e < a.heads * (a.p - a.vdim); e += THREADS) {
-                const int h = e / (a.p - a.vdim);
-                out[h * a.p + a.vdim + e - h * (a.p - a.vdim)] = from_f32<T>(0.f);
-            }
+    auto gate = [&](int c) {
+        const float u = to_f32(g[c]);
+        return u * sigmoid_for<T>(u);
+    };
+    float s = 0.f;
+    for (int e = part * a.part + threadIdx.x; e < (part + 1) * a.part; e += 256) {
+        const int c = at(e);
+        const float v = to_f32(x[c]) * (a.weight ? gate(c) : 1.f);
+        s = fmaf(v, v, s);
     }
+    s = block_sum(s, red);
+    const float rs = 1.0f / sqrtf(s / (float)a.part + (float)a.eps);
+    for (int e = part * a.part + threadIdx.x; e < (part + 1) * a.part; e += 256) {
+        const int c = at(e);
+        out[c] = from_f32<T>(to_f32(x[c]) * gate(c) * rs * (a.weight ? a.weight[c] : a.scale));
+    }
+    if (part == 0 && a.p > a.vdim)                       // padding of every head
+        for (int e = threadIdx.x; e < a.heads * (a.p - a.vdim); e += 256) {
+            const int h = e / (a.p - a.vdim);
+            out[h * a.p + a.vdim + e - h * (a.p - a.vdim)] = from_f32<T>(0.f);
+        }
+}
+
+template <typename T, bool FIRST>
+int gated_norm_packed(const zkfp_gated_norm_args& a, int parts, int stride, cudaStream_t st)
+{
+    const long long units = a.rows * parts;
+    if (units > 0x7fffffffll) return ZKDS_ERR_UNSUPPORTED;
+    const unsigned warps = (unsigned)((units + 7) / 8);
+    if (stride <= 256) gated_norm_kernel<T, 32, 1, FIRST><<<warps, 256, 0, st>>>(a, parts, stride);
+    else if (stride <= 512) gated_norm_kernel<T, 32, 2, FIRST><<<warps, 256, 0, st>>>(a, parts, stride);
+    else if (stride <= 1024) gated_norm_kernel<T, 32, 4, FIRST><<<warps, 256, 0, st>>>(a, parts, stride);
+    else if (stride <= 2048) gated_norm_kernel<T, 32, 8, FIRST><<<warps, 256, 0, st>>>(a, parts, stride);
+    else gated_norm_kernel<T, 256, 4, FIRST><<<(unsigned)units, 256, 0, st>>>(a, parts, stride);
+    return fp_launched();
 }
 
 template <typename T>
 int gated_norm(const zkfp_gated_norm_args& a, cudaStream_t st)
 {
     const bool whole_head = a.part == a.vdim;
-    const bool packed = whole_head || (a.p == a.vdim && a.part % 8 == 0);
     const int parts = a.heads * a.vdim / a.part, stride = whole_head ? a.p : a.part;
-    const bool wide = a.part > 512;
-    const long long per = wide ? 1 : 8, blocks = (a.rows * parts + per - 1) / per;
-    if (blocks > 0x7fffffffll) return ZKDS_ERR_UNSUPPORTED;
-    if (packed && wide) gated_norm_kernel<T, 256, true><<<(unsigned)blocks, 256, 0, st>>>(a, parts, stride);
-    else if (packed) gated_norm_kernel<T, 32, true><<<(unsigned)blocks, 256, 0, st>>>(a, parts, stride);
-    else if (wide) gated_norm_kernel<T, 256, false><<<(unsigned)blocks, 256, 0, st>>>(a, parts, stride);
-    else gated_norm_kernel<T, 32, false><<<(unsigned)blocks, 256, 0, st>>>(a, parts, stride);
+    if (whole_head || (a.p == a.vdim && a.part % 8 == 0))
+        return a.weight ? gated_norm_packed<T, true>(a, parts, stride, st) : gated_norm_packed<T, false>(a, parts, stride, st);
+    if (a.rows * parts > 0x7fffffffll) return ZKDS_ERR_UNSUPPORTED;
+    gated_norm_any_kernel<T><<<(unsigned)(a.rows * parts), 256, 0, st>>>(a, parts);
     return fp_launched();
 }
 

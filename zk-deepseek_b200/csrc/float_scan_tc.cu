@@ -58,7 +58,7 @@ struct ScanTcParams {
     long long step_tok, n_slots;
     int seq, heads, heads_per_qk, n, p, segq, chunks, chunks_per_segment, segments;
     float k_scale;
-    uint32_t smem_bytes;
+    uint32_t smem_bytes[2];                    // without and with outputs
     int* error_flag;
 };
 
@@ -68,9 +68,10 @@ struct ChunkDecays {
     float col[kL - 32];                        // decay from a token to the end of its block of 32, times its weight
 };
 
+template <int STAGES>
 struct ScanTcShared {
-    ChunkDecays d[2];
-    uint64_t qk_full[2], qk_empty[2], v_full[2], v_empty[2], out_full[2], vp_full[2], ds_full[2], s_full, p_full, st_full, qs_full, o_full;
+    ChunkDecays d[STAGES];
+    uint64_t qk_full[STAGES], qk_empty[STAGES], v_full[STAGES], v_empty[STAGES], out_full[2], vp_full[2], ds_full[2], s_full, p_full, st_full, o_full;
     uint32_t tmem;
     int abort;
 };
@@ -123,10 +124,14 @@ scan_decay_kernel(const ScanTcParams p)
     __shared__ float raw[kL][33];
     const int c = blockIdx.x, h0 = blockIdx.y * 32, b = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (p.step) {
-        for (int i = warp; i < kL; i += 8) {
-            const int t = c * kL + i;
-            raw[i][lane] = t < p.seq && h0 + lane < p.heads ? p.step[((long long)b * p.seq + t) * p.step_tok + h0 + lane] : 0.f;
+        float v[kL / 8];                           // all loads in flight
+#pragma unroll
+        for (int i = 0; i < kL / 8; ++i) {
+            const int t = c * kL + i * 8 + warp;
+            v[i] = t < p.seq && h0 + lane < p.heads ? p.step[((long long)b * p.seq + t) * p.step_tok + h0 + lane] : 0.f;
         }
+#pragma unroll
+        for (int i = 0; i < kL / 8; ++i) raw[i * 8 + warp][lane] = v[i];
         __syncthreads();
     }
     for (int k = 0; k < 4; ++k) {
@@ -183,14 +188,15 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int rows_s = p.segq * 64;                                       // rows of the state tiles
     const uint32_t bytes_q = OUT ? (uint32_t)p.segq * kSegB : 0u, stage_bytes = bytes_q + 3 * kSegB;
     const uint32_t bytes_s = (uint32_t)rows_s * 128u;
-    // without outputs there is room for a second pair of value tiles instead of the state's
-    const uint32_t tile_bytes = 2 * stage_bytes + (OUT ? 2 * kSegB + 2 * bytes_s : 4 * kSegB), vp_step = OUT ? 0u : 2 * kSegB;
-    if (base + tile_bytes + sizeof(ScanTcShared) > raw + p.smem_bytes) {  // not the alignment the host counted on
+    // without outputs there is room for a third stage, and for a second pair of value tiles instead of the state's
+    constexpr int kStages = OUT ? 2 : 3;
+    const uint32_t tile_bytes = kStages * stage_bytes + (OUT ? 2 * kSegB + 2 * bytes_s : 4 * kSegB), vp_step = OUT ? 0u : 2 * kSegB;
+    if (base + tile_bytes + sizeof(ScanTcShared<kStages>) > raw + p.smem_bytes[OUT]) {  // not the alignment the host counted on
         if (threadIdx.x == 0) *(volatile int*)p.error_flag = 1;
         return;
     }
-    ScanTcShared& s = *reinterpret_cast<ScanTcShared*>(base + tile_bytes);
-    uint8_t* vp = base + 2 * stage_bytes;                                 // scaled values: rounded, remainder
+    ScanTcShared<kStages>& s = *reinterpret_cast<ScanTcShared<kStages>*>(base + tile_bytes);
+    uint8_t* vp = base + kStages * stage_bytes;                                 // scaled values: rounded, remainder
     uint8_t* st = vp + 2 * kSegB;                                         // state: rounded, remainder
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int slice = blockIdx.x, head = blockIdx.y, b = blockIdx.z / p.segments, seg = blockIdx.z % p.segments;
@@ -202,11 +208,13 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 
     if (threadIdx.x == 0) {
         s.abort = 0;
-        for (int i = 0; i < 2; ++i) {
+        for (int i = 0; i < kStages; ++i) {
             mbar_init(smem_u32(&s.qk_full[i]), 1);
             mbar_init(smem_u32(&s.qk_empty[i]), 1);
             mbar_init(smem_u32(&s.v_full[i]), 1);
             mbar_init(smem_u32(&s.v_empty[i]), OUT ? kElemWarps : 1);
+        }
+        for (int i = 0; i < 2; ++i) {
             mbar_init(smem_u32(&s.out_full[i]), kElemWarps);
             mbar_init(smem_u32(&s.vp_full[i]), kElemWarps);
             mbar_init(smem_u32(&s.ds_full[i]), 1);
@@ -214,8 +222,7 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         mbar_init(smem_u32(&s.s_full), 1);
         mbar_init(smem_u32(&s.p_full), kElemWarps);
         mbar_init(smem_u32(&s.st_full), kElemWarps);
-        mbar_init(smem_u32(&s.qs_full), 1);
-        mbar_init(smem_u32(&s.o_full), 1);
+        mbar_init(smem_u32(&s.o_full), 2);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncwarp();
@@ -225,13 +232,17 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     tc_fence_after();
     const uint32_t tmem = s.tmem;
 
+    // stage of chunk c, and how often that stage has been used before
+    auto stage_of = [](int c) { return OUT ? c & 1 : c % 3; };
+    auto turn_of = [](int c) { return OUT ? c >> 1 : c / 3; };
+
     if (warp == kElemWarps + 1) {
         if (lane == 0) {
             const int hq = head / p.heads_per_qk;
             const ChunkDecays* decays = reinterpret_cast<const ChunkDecays*>(p.decays) + ((long long)b * p.heads + head) * p.chunks + c_begin;
             for (int c = 0; c < nc; ++c) {
-                const int stage = c & 1, y = b * p.seq + (c_begin + c) * kL;
-                const uint32_t free_phase = (uint32_t)((c >> 1) & 1) ^ 1u, dst = smem0 + (uint32_t)stage * stage_bytes;
+                const int stage = stage_of(c), y = b * p.seq + (c_begin + c) * kL;
+                const uint32_t free_phase = (uint32_t)(turn_of(c) & 1) ^ 1u, dst = smem0 + (uint32_t)stage * stage_bytes;
                 if (!mbar_wait_polling(smem_u32(&s.v_empty[stage]), free_phase, abort_flag)) break;
                 uint32_t bar = smem_u32(&s.v_full[stage]);
                 mbar_expect_tx(bar, kSegB + (uint32_t)sizeof(ChunkDecays));
@@ -284,8 +295,8 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             }
         } else {
             for (int c = 0; c < nc; ++c) {
-                const uint32_t q = smem0 + (uint32_t)(c & 1) * stage_bytes;
-                if (!wait(&s.qk_full[c & 1], c >> 1) || !wait(&s.vp_full[c & 1], c >> 1)) break;
+                const uint32_t q = smem0 + (uint32_t)stage_of(c) * stage_bytes;
+                if (!wait(&s.qk_full[stage_of(c)], turn_of(c)) || !wait(&s.vp_full[c & 1], c >> 1)) break;
                 const uint64_t vd = smem_desc_mn_sw128(smem_u32(vp) + (uint32_t)(c & 1) * vp_step, kSegB);
                 const uint32_t d = tmem + kColD - (OUT ? 0u : (uint32_t)(c & 1) * 128u);
                 const uint64_t kd = smem_desc_mn_sw128(q + bytes_q, kSegB);
@@ -295,8 +306,8 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         umma_bf16(d, kd + (uint64_t)(k * 128), vd + (uint64_t)(k * 128), idesc_d, k ? 1u : 0u);
                     umma_commit(smem_u32(&s.ds_full[c & 1]));
                     if (!OUT) {
-                        umma_commit(smem_u32(&s.qk_empty[c & 1]));
-                        umma_commit(smem_u32(&s.v_empty[c & 1]));
+                        umma_commit(smem_u32(&s.qk_empty[stage_of(c)]));
+                        umma_commit(smem_u32(&s.v_empty[stage_of(c)]));
                     }
                 }
                 if (!OUT) continue;
@@ -308,7 +319,7 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         if (k < steps)
                             umma_bf16(tmem + kColQS, smem_desc_sw128(q + (uint32_t)(k >> 2) * kSegB + (uint32_t)(k & 3) * 32u),
                                       smem_desc_mn_sw128(smem_u32(st) + (uint32_t)k * 2048u, bytes_s), idesc_s, k ? 1u : 0u);
-                    umma_commit(smem_u32(&s.qs_full));
+                    umma_commit(smem_u32(&s.o_full));
                 }
             }
         }
@@ -328,18 +339,22 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const int part = warp >> 2, quarter = warp & 3, row = quarter * 32 + lane;
         const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
         const int col0 = slice * kPT + part * 16;
-        const bool fresh = p.start[b] == 0;
-        const long long sh = ((long long)b * p.heads + head) * p.segments + seg;
-        float* state = p.state + ((slot * p.heads + head) * p.n + row) * p.p + col0;
-        float* seg_state = p.seg_state + (sh * p.n + row) * p.p + col0;
-        const float* from = !OUT ? nullptr : p.segments > 1 ? seg_state : fresh ? nullptr : state;
+        // this thread's 16 values of the state in global memory
+        auto state_at = [&](bool own) {
+            const long long sh = ((long long)b * p.heads + head) * p.segments + seg;
+            return own ? p.state + ((slot * p.heads + head) * p.n + row) * p.p + col0 : p.seg_state + (sh * p.n + row) * p.p + col0;
+        };
         float S[16];
+        {
+            const bool segmented = p.segments > 1, read = OUT && row < p.n && (segmented || p.start[b] != 0);
+            const float* from = state_at(!segmented);
 #pragma unroll
-        for (int i = 0; i < 16; i += 8) {
-            float v[8] = {};
-            if (from && row < p.n && col0 + i < p.p) load8(from + i, v);
+            for (int i = 0; i < 16; i += 8) {
+                float v[8] = {};
+                if (read && col0 + i < p.p) load8(from + i, v);
 #pragma unroll
-            for (int k = 0; k < 8; ++k) S[i + k] = v[k];
+                for (int k = 0; k < 8; ++k) S[i + k] = v[k];
+            }
         }
         auto arrive = [&](uint64_t* bar) {
             tc_fence_before();
@@ -351,15 +366,15 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             arrive(bar);
         };
         auto wait = [&](uint64_t* bar, int phase) { return mbar_wait_polling(smem_u32(bar), (uint32_t)(phase & 1), abort_flag); };
-        auto value_tile = [&](int c) { return base + (uint32_t)(c & 1) * stage_bytes + bytes_q + 2 * kSegB; };
+        auto value_tile = [&](int c) { return base + (uint32_t)stage_of(c) * stage_bytes + bytes_q + 2 * kSegB; };
         // values scaled by what is left of them at the chunk's end
         float l_row = 0.f, l_end = 0.f, l_row_next, l_end_next;          // a stage may be refilled once its values are scaled
         auto scale_values = [&](int c) {
             float v[16];
             load_row(value_tile(c), row, part, v);
-            l_row_next = s.d[c & 1].l[row];
-            l_end_next = s.d[c & 1].l[kL - 1];
-            const float f = exp2_fast(l_end_next - s.d[c & 1].lw[row]);
+            l_row_next = s.d[stage_of(c)].l[row];
+            l_end_next = s.d[stage_of(c)].l[kL - 1];
+            const float f = exp2_fast(l_end_next - s.d[stage_of(c)].lw[row]);
 #pragma unroll
             for (int i = 0; i < 16; ++i) v[i] *= f;
             uint8_t* dst = vp + (uint32_t)(c & 1) * vp_step;
@@ -379,6 +394,29 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             l_row = l_row_next;
             l_end = l_end_next;
             if (OUT) {
+                // what is left at each row of each column's weight, half of it while the scores are on their way
+                const float f = part < quarter ? exp2_fast(l_row - s.d[stage].l[part * 32 + 31]) : 0.f;
+                float g[16];
+                auto factors = [&](int q) {
+                    if (part < quarter) {
+#pragma unroll
+                        for (int i = 0; i < 16; i += 4) {
+                            const float4 x = *reinterpret_cast<const float4*>(&s.d[stage].col[part * 32 + q * 16 + i]);
+                            g[i] = f * x.x; g[i + 1] = f * x.y; g[i + 2] = f * x.z; g[i + 3] = f * x.w;
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 16; i += 4) {
+                            const float4 x = *reinterpret_cast<const float4*>(&s.d[stage].lw[part * 32 + q * 16 + i]);
+                            const int e = q * 16 + i;
+                            g[i] = e <= lane ? exp2_fast(l_row - x.x) : 0.f;
+                            g[i + 1] = e + 1 <= lane ? exp2_fast(l_row - x.y) : 0.f;
+                            g[i + 2] = e + 2 <= lane ? exp2_fast(l_row - x.z) : 0.f;
+                            g[i + 3] = e + 3 <= lane ? exp2_fast(l_row - x.w) : 0.f;
+                        }
+                    }
+                };
+                if (part <= quarter) factors(0);
                 if (!(ok = wait(&s.s_full, c))) break;
                 tc_fence_after();
                 uint32_t w[16];
@@ -386,38 +424,22 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
                     for (int i = 0; i < 16; ++i) w[i] = 0u;
                 } else {
-                    float v[32];
-                    tmem_ld32(tmem + kColS + lanes + (uint32_t)part * 32u, v);
-                    if (part < quarter) {
-                        const float f = exp2_fast(l_row - s.d[stage].l[part * 32 + 31]);
+                    const uint32_t ts = tmem + kColS + lanes + (uint32_t)part * 32u;
+#pragma unroll
+                    for (int q = 0; q < 2; ++q) {
+                        float v[16];
+                        tmem_ld16f(ts + (uint32_t)(q * 16), v);
+                        if (q) factors(1);
                         tmem_ld_wait();
 #pragma unroll
-                        for (int i = 0; i < 32; i += 4) {
-                            const float4 g = *reinterpret_cast<const float4*>(&s.d[stage].col[part * 32 + i]);
-                            v[i] *= f * g.x;
-                            v[i + 1] *= f * g.y;
-                            v[i + 2] *= f * g.z;
-                            v[i + 3] *= f * g.w;
-                        }
-                    } else {
-                        tmem_ld_wait();
-#pragma unroll
-                        for (int i = 0; i < 32; i += 4) {
-                            const float4 g = *reinterpret_cast<const float4*>(&s.d[stage].lw[part * 32 + i]);
-                            v[i] = i <= lane ? v[i] * exp2_fast(l_row - g.x) : 0.f;
-                            v[i + 1] = i + 1 <= lane ? v[i + 1] * exp2_fast(l_row - g.y) : 0.f;
-                            v[i + 2] = i + 2 <= lane ? v[i + 2] * exp2_fast(l_row - g.z) : 0.f;
-                            v[i + 3] = i + 3 <= lane ? v[i + 3] * exp2_fast(l_row - g.w) : 0.f;
-                        }
+                        for (int i = 0; i < 8; ++i) w[q * 8 + i] = pack_bf16(v[2 * i] * g[2 * i], v[2 * i + 1] * g[2 * i + 1]);
                     }
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) w[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
                 }
                 tmem_st16(tmem + kColP + lanes + (uint32_t)part * 16u, w);
                 tmem_st_wait();
                 arrive(&s.p_full);
             }
-            auto next_values = [&] { return c + 1 == nc || wait(&s.v_full[stage ^ 1], (c + 1) >> 1); };
+            auto next_values = [&] { return c + 1 == nc || wait(&s.v_full[stage_of(c + 1)], turn_of(c + 1)); };
             if (!OUT) {
                 if (!(ok = next_values())) break;
                 if (c + 1 < nc) scale_values(c + 1);
@@ -441,17 +463,20 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 scale_values(c + 1);
             }
             if (OUT) {
-                if (!(ok = wait(&s.qs_full, c) && wait(&s.o_full, c))) break;
+                if (!(ok = wait(&s.o_full, c))) break;
                 tc_fence_after();
-                float o[16], x[16], r[16];
-                tmem_ld16f(tmem + kColO + lanes + (uint32_t)part * 16u, o);
-                tmem_ld16f(tmem + kColQS + lanes + (uint32_t)part * 16u, x);
-                tmem_ld16f(tmem + kColQS + lanes + 64u + (uint32_t)part * 16u, r);
+                float o[16], x[16];
+                tmem_ld16f(tmem + kColQS + lanes + (uint32_t)part * 16u, o);
+                tmem_ld16f(tmem + kColQS + lanes + 64u + (uint32_t)part * 16u, x);
                 const float f = exp2_fast(l_row);
                 uint8_t* tile = base + (uint32_t)stage * stage_bytes;
                 tmem_ld_wait();
 #pragma unroll
-                for (int i = 0; i < 16; ++i) o[i] = fmaf(f, x[i] + r[i], o[i]);
+                for (int i = 0; i < 16; ++i) o[i] = f * (o[i] + x[i]);
+                tmem_ld16f(tmem + kColO + lanes + (uint32_t)part * 16u, x);
+                tmem_ld_wait();
+#pragma unroll
+                for (int i = 0; i < 16; ++i) o[i] += x[i];
                 if (p.skip) {
                     load_row(value_tile(c), row, part, x);
 #pragma unroll
@@ -470,8 +495,8 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 if (lane == 0 && c + 1 < nc) mbar_arrive(smem_u32(&s.st_full));
             }
         }
-        float* to = OUT ? (seg == p.segments - 1 ? state : nullptr) : seg_state;
-        if (to && row < p.n) {
+        if ((!OUT || seg == p.segments - 1) && row < p.n) {
+            float* to = state_at(OUT);
 #pragma unroll
             for (int i = 0; i < 16; i += 8)
                 if (col0 + i < p.p) {
@@ -481,7 +506,7 @@ scan_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     store8(to + i, y);
                 }
         }
-        if (!OUT && slice == 0 && threadIdx.x == 0) p.seg_decay[sh] = total;
+        if (!OUT && slice == 0 && threadIdx.x == 0) p.seg_decay[((long long)b * p.heads + head) * p.segments + seg] = total;
     }
     tc_fence_before();
     __syncthreads();
@@ -501,20 +526,31 @@ scan_segments_kernel(const ScanTcParams p)
     float4 run = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.start[b] != 0) run = *reinterpret_cast<const float4*>(p.state + (slot * p.heads + head) * size + i);
     const long long sh = ((long long)b * p.heads + head) * p.segments;
-    for (int s = 0; s < p.segments; ++s) {
-        float4* at = reinterpret_cast<float4*>(p.seg_state + (sh + s) * size + i);
-        const float4 mine = *at;
-        const float f = exp2_fast(p.seg_decay[sh + s]);
-        *at = run;
-        run.x = fmaf(f, run.x, mine.x); run.y = fmaf(f, run.y, mine.y);
-        run.z = fmaf(f, run.z, mine.z); run.w = fmaf(f, run.w, mine.w);
+    constexpr int B = 4;                           // segments whose states are loaded together
+    for (int s0 = 0; s0 < p.segments; s0 += B) {
+        float4 mine[B];
+        float f[B];
+#pragma unroll
+        for (int k = 0; k < B; ++k)
+            if (s0 + k < p.segments) {
+                mine[k] = *reinterpret_cast<const float4*>(p.seg_state + (sh + s0 + k) * size + i);
+                f[k] = exp2_fast(p.seg_decay[sh + s0 + k]);
+            }
+#pragma unroll
+        for (int k = 0; k < B; ++k)
+            if (s0 + k < p.segments) {
+                *reinterpret_cast<float4*>(p.seg_state + (sh + s0 + k) * size + i) = run;
+                run.x = fmaf(f[k], run.x, mine[k].x); run.y = fmaf(f[k], run.y, mine[k].y);
+                run.z = fmaf(f[k], run.z, mine[k].z); run.w = fmaf(f[k], run.w, mine[k].w);
+            }
     }
 }
 
-size_t scan_smem(int n)
+size_t scan_smem(int n, bool out)
 {
     const size_t segq = (size_t)(n + 63) / 64;
-    const size_t bytes = 2 * (segq + 3) * kSegB + 2 * kSegB + 2 * segq * 64 * 128 + sizeof(ScanTcShared) + 128;
+    const size_t tiles = out ? 2 * (segq + 3) * kSegB + 2 * kSegB + 2 * segq * 64 * 128 : 3 * 3 * kSegB + 4 * kSegB;
+    const size_t bytes = tiles + (out ? sizeof(ScanTcShared<2>) : sizeof(ScanTcShared<3>)) + 64;
     return bytes + 1024 < kScanSmemAll ? bytes + 1024 : kScanSmemAll;
 }
 
@@ -578,7 +614,7 @@ int launch_scan_tc(const zkfp_scan_args& a, cudaStream_t st)
     if (!fp_tensor_map(&q, a.q, 3, dqk, sq, box) || !fp_tensor_map(&k, a.k, 3, dqk, sk, box) || !fp_tensor_map(&v, a.v, 3, dv, sv, box) ||
         !fp_tensor_map(&o, a.out, 4, dout, so, box_o))
         return ZKDS_ERR_UNSUPPORTED;
-    p.smem_bytes = (uint32_t)scan_smem(a.n);
+    for (int i = 0; i < 2; ++i) p.smem_bytes[i] = (uint32_t)scan_smem(a.n, i);
     const dim3 grid((unsigned)((a.p + kPT - 1) / kPT), (unsigned)a.heads, (unsigned)(a.batch * p.segments));
     if (grid.z > 65535u) return ZKDS_ERR_UNSUPPORTED;
     scan_decay_kernel<<<dim3((unsigned)p.chunks, (unsigned)((a.heads + 31) / 32), (unsigned)a.batch), 256, 0, st>>>(p);
@@ -586,7 +622,7 @@ int launch_scan_tc(const zkfp_scan_args& a, cudaStream_t st)
     if (rc != ZKDS_OK) return rc;
     if (p.segments > 1) {
         ZKDS_CUDA(cudaFuncSetAttribute(scan_chunk_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kScanSmemAll));
-        scan_chunk_kernel<false><<<grid, kScanThreads, p.smem_bytes, st>>>(q, k, v, o, p);
+        scan_chunk_kernel<false><<<grid, kScanThreads, p.smem_bytes[0], st>>>(q, k, v, o, p);
         rc = fp_launched();
         if (rc != ZKDS_OK) return rc;
         scan_segments_kernel<<<dim3((unsigned)((a.n * a.p + 1023) / 1024), (unsigned)a.heads, (unsigned)a.batch), 256, 0, st>>>(p);
@@ -594,7 +630,7 @@ int launch_scan_tc(const zkfp_scan_args& a, cudaStream_t st)
         if (rc != ZKDS_OK) return rc;
     }
     ZKDS_CUDA(cudaFuncSetAttribute(scan_chunk_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kScanSmemAll));
-    scan_chunk_kernel<true><<<grid, kScanThreads, p.smem_bytes, st>>>(q, k, v, o, p);
+    scan_chunk_kernel<true><<<grid, kScanThreads, p.smem_bytes[1], st>>>(q, k, v, o, p);
     return fp_launched();
 }
 

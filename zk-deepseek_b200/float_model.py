@@ -259,7 +259,7 @@ class StackedMixer(nn.Module):
         t = t.view((heads, size) + t.shape[1:])
         if order is not None:
             t = t[:, order]
-        out = torch.zeros((heads, pad) + t.shape[2:], dtype=t.dtype)
+        out = torch.zeros((heads, pad) + t.shape[2:], dtype=t.dtype, device=t.device)
         out[:, :size] = t
         return out.view((heads * pad,) + t.shape[2:])
 
